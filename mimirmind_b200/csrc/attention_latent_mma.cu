@@ -5,6 +5,9 @@
 //   s_j = (q . row_j) * scale;  p = softmax_j over the keys j <= position (and inside the window, if one is given);
 //   o = sum_j p_j row_j[0 : rank]
 //
+// With a sink (one number per head) the softmax's denominator also holds exp(sink_h): it starts the running maximum and
+// mass of the first split's rows.
+//
 // One CTA (8 or 16 warps: 2 or 4 row groups of 4 warps) owns a tile of 32 or 64 query rows, each row one (token, head)
 // pair of one request; because every head reads the same keys, a key tile is fetched once for all of them.  Keys stream through shared memory in tiles of 32,
 // gathered page by page with cp.async, two stages deep.  Per key tile:
@@ -66,7 +69,7 @@ __global__ void __launch_bounds__(RG * 128) attention_latent_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool, __nv_bfloat16* __restrict__ out,
     float* __restrict__ out32, float* __restrict__ part_o, float* __restrict__ part_ml, const int32_t* __restrict__ tiles,
     const int32_t* __restrict__ positions, const int32_t* __restrict__ block_table, int table_width, int page_size, int H,
-    int wide, int rank, int window, float scale_log2) {
+    int wide, int rank, int window, float scale_log2, const float* __restrict__ sink) {
     constexpr int THREADS = RG * 128;             // RG row groups x 4 column groups of one warp each
     constexpr int ROWS = 16 * MT * RG;            // query rows of the CTA
     constexpr int TPR = THREADS / ROWS;           // threads per row in the softmax stage
@@ -125,6 +128,10 @@ __global__ void __launch_bounds__(RG * 128) attention_latent_kernel(
     // the softmax stage: thread t holds row t / TPR and the keys (t % TPR) * KPT .. + KPT - 1 of a tile
     const int srow = threadIdx.x / TPR, skey = (threadIdx.x % TPR) * KPT;
     float m_run = -INFINITY, l_run = 0.0f;
+    if (sink != nullptr && split == 0 && srow < n_rows) {
+        m_run = sink[head0 + srow % n_heads] * LAT_LOG2E;
+        l_run = 1.0f;
+    }
     const int col0 = cg * NT * 8;                    // this warp's first value column
     const int id = lane >> 3, rr = lane & 7;
 
@@ -316,9 +323,9 @@ static size_t latent_smem(int wide, int rows) {
 
 #define LAT_ARGS const void* q, const void* pool, void* out, void* part_o, void* part_ml, int n_splits, const void* tiles, \
                  int n_tiles, int n_rows, const void* positions, const void* table, int table_width, int page_size, int H, \
-                 int wide, int rank, int window, float scale, int out_f32, cudaStream_t s
+                 int wide, int rank, int window, float scale, const void* sink, int out_f32, cudaStream_t s
 #define LAT_PASS q, pool, out, part_o, part_ml, n_splits, tiles, n_tiles, n_rows, positions, table, table_width, page_size, H, \
-                 wide, rank, window, scale, out_f32, s
+                 wide, rank, window, scale, sink, out_f32, s
 
 template <int NT, int MT, int RG>
 static int launch_latent(LAT_ARGS) {
@@ -336,7 +343,7 @@ static int launch_latent(LAT_ARGS) {
     mm_launch(kernel, dim3(n_tiles, n_splits), dim3(RG * 128), smem, s, (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool,
               out_f32 ? nullptr : (__nv_bfloat16*)out, out_f32 ? (float*)out : nullptr, (float*)part_o, (float*)part_ml,
               (const int32_t*)tiles, (const int32_t*)positions, (const int32_t*)table, table_width, page_size, H, wide, rank, window,
-              scale * LAT_LOG2E);
+              scale * LAT_LOG2E, (const float*)sink);
     MM_CHECK_LAUNCH();
     if (n_splits > 1) {
         mm_launch(attention_latent_merge_kernel, dim3(n_rows), dim3(rank >= 256 ? 128 : 64), 0, s, out_f32 ? nullptr : (__nv_bfloat16*)out,
@@ -358,11 +365,11 @@ MM_EXPORT int mm_attention_latent_tile_rows(int wide) { return latent_smem(wide,
 
 // q [n, H, wide] and pool [pages, page, wide] bfloat16; out [n, H, rank] bfloat16 or fp32.  tiles int32 [n_tiles, 5] of at
 // most tile_rows (32 or 64) rows each; n_rows = n * H.  n_splits > 1: part_o [n_rows, n_splits, rank] and part_ml
-// [n_rows, n_splits, 2] (fp32).
+// [n_rows, n_splits, 2] (fp32).  sink: fp32 [H] or null.
 MM_EXPORT int mm_attention_latent_bf16(const void* q, const void* pool, void* out, void* part_o, void* part_ml, int n_splits,
                                        const void* tiles, int n_tiles, int tile_rows, int n_rows, const void* positions,
                                        const void* table, int table_width, int page_size, int H, int wide, int rank, int window,
-                                       float scale, int out_f32, void* stream) {
+                                       float scale, const void* sink, int out_f32, void* stream) {
     MM_REQUIRE(mm_attention_latent_supported(wide, rank), "latent attention: rank a multiple of 16 up to 512, row width a multiple of 8");
     MM_REQUIRE(tile_rows == 32 || (tile_rows == 64 && mm_attention_latent_tile_rows(wide) == 64), "latent attention: tiles of 32 or 64 rows");
     MM_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (part_o != nullptr && part_ml != nullptr)),

@@ -2,11 +2,11 @@
 //
 //   * rope_half_table: (cos, sin) per (token, frequency) of position * frequency, the frequency given as the sum of two
 //     floats (made in float64 on the host) and the product's rounding error carried into the result, so that the angle
-//     is as good as a float64 product although every operation is a 32-bit one;
+//     is as good as a float64 product although every operation is a 32-bit one; a factor may multiply both;
 //   * qkv_split_post: fp32 rows of a projection (after their convolution, if any) cut into queries, keys and values; the
 //     queries go to a dense buffer, keys and values into their pages, in the run's dtype;
 //   * latent_prep: the step between the projections of a latent attention and its kernel: the latent vector is RMS-normed,
-//     the shared rotated key part and every head's rotated query part are turned (pairs i, i + dims/2), and latent and
+//     the shared rotated key part and every head's rotated query part are turned (pairs i, i + dims/2, or 2i, 2i + 1), and latent and
 //     rotated key are written side by side into one per-token cache array;
 //   * head_matmul: out[t, h, :] = in[t, h, :] . M[h] with a matrix per head (absorbing the key or value up-projection
 //     of a latent attention into the query or the output), fp32 FMAs over eight runs of k, summed in order;
@@ -16,7 +16,7 @@
 
 // ---------------------------------------------------------------------------------------------------------------
 __global__ void rope_half_table_kernel(const int32_t* __restrict__ positions, const float* __restrict__ f_hi, const float* __restrict__ f_lo,
-                                       float2* __restrict__ table, int n_tokens, int half) {
+                                       float2* __restrict__ table, int n_tokens, int half, float factor) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (long long)n_tokens * half) return;
     const int t = (int)(i / half), p = (int)(i - (long long)t * half);
@@ -25,15 +25,15 @@ __global__ void rope_half_table_kernel(const int32_t* __restrict__ positions, co
     const float rest = fmaf(pos, f_lo[p], fmaf(pos, f_hi[p], -a));     // what the rounded product left out, and the low word's share
     float sn, cs;
     sincosf(a, &sn, &cs);
-    table[i] = make_float2(fmaf(-rest, sn, cs), fmaf(rest, cs, sn));
+    table[i] = make_float2(fmaf(-rest, sn, cs) * factor, fmaf(rest, cs, sn) * factor);
 }
 
-MM_EXPORT int mm_rope_half_table(const void* positions, const void* f_hi, const void* f_lo, void* table, int n_tokens, int half, void* stream) {
+MM_EXPORT int mm_rope_half_table(const void* positions, const void* f_hi, const void* f_lo, void* table, int n_tokens, int half, float factor, void* stream) {
     MM_REQUIRE(n_tokens >= 0 && half > 0, "rotation table: bad sizes");
     if (n_tokens == 0) return MM_OK;
     const long long total = (long long)n_tokens * half;
     mm_launch(rope_half_table_kernel, dim3(ceil_div(total, 256)), dim3(256), 0, (cudaStream_t)stream, (const int32_t*)positions,
-              (const float*)f_hi, (const float*)f_lo, (float2*)table, n_tokens, half);
+              (const float*)f_hi, (const float*)f_lo, (float2*)table, n_tokens, half, factor);
     MM_CHECK_LAUNCH();
     return MM_OK;
 }
@@ -85,17 +85,29 @@ MM_EXPORT int mm_qkv_split_post(const void* rows, int ld, int q_off, int k_off, 
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// rows [n, ld] fp32: H heads of (dk plain, dr rotated) query numbers at q_off; the latent's `rank` numbers and the shared
-// key part's dr numbers at c_off.  rot [n, rot_dims / 2] (cos, sin); dimensions from rot_dims on of a rotated part pass.
+// q_rows [n, ldq] fp32: H heads of (dk plain, dr rotated) query numbers at q_off; c_rows [n, ldc] fp32 (may be the same
+// rows): the latent's `rank` numbers and the shared key part's dr numbers at c_off.  rot [n, rot_dims / 2] (cos, sin);
+// number i turns with i + rot_dims / 2, or with `pairs` 2i with 2i + 1; numbers from rot_dims on of a rotated part pass.
 // q_plain [n, H, dk]; q_full [n, H, rank + dr] gets each head's rotated part at [rank, rank + dr); pages
 // [pages, 1, page_size, rank + dr] get (normed latent, rotated key part).
+__device__ __forceinline__ float turned(const float* part, const float2* rt, int e, int rot_dims, int pairs) {
+    if (e >= rot_dims) return part[e];
+    const int half = rot_dims >> 1;
+    const int f = pairs ? e >> 1 : (e < half ? e : e - half);                     // the pair's frequency
+    const bool first = pairs ? (e & 1) == 0 : e < half;
+    const float other = part[pairs ? e ^ 1 : (first ? e + half : e - half)];
+    return first ? part[e] * rt[f].x - other * rt[f].y : part[e] * rt[f].x + other * rt[f].y;
+}
+
 template <typename T>
-__global__ void latent_prep_kernel(const float* __restrict__ rows, int ld, int q_off, int c_off, const void* __restrict__ norm_w, int w_dtype,
-                                   float eps, const float2* __restrict__ rot, int rot_dims, T* __restrict__ q_plain, T* __restrict__ q_full,
-                                   T* __restrict__ pages, const int32_t* __restrict__ slots, int page_size, int H, int dk, int dr, int rank) {
+__global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, int q_off, const float* __restrict__ c_rows, int ldc, int c_off,
+                                   const void* __restrict__ norm_w, int w_dtype, float eps, const float2* __restrict__ rot, int rot_dims, int pairs,
+                                   T* __restrict__ q_plain, T* __restrict__ q_full, T* __restrict__ pages, const int32_t* __restrict__ slots,
+                                   int page_size, int H, int dk, int dr, int rank) {
     __shared__ float scratch[32];
     const int t = blockIdx.x;
-    const float* row = rows + (size_t)t * ld;
+    const float* row = q_rows + (size_t)t * ldq;
+    const float* crow = c_rows + (size_t)t * ldc;
     const int half = rot_dims / 2;
     const float2* rt = rot + (size_t)t * half;
     const int wide = rank + dr;
@@ -106,18 +118,11 @@ __global__ void latent_prep_kernel(const float* __restrict__ rows, int ld, int q
     }
     for (int i = threadIdx.x; i < H * dr; i += blockDim.x) {
         const int h = i / dr, e = i - h * dr;
-        const float* part = row + q_off + h * (dk + dr) + dk;
-        float v = part[e];
-        if (e < half) {
-            v = part[e] * rt[e].x - part[e + half] * rt[e].y;
-        } else if (e < rot_dims) {
-            v = part[e] * rt[e - half].x + part[e - half] * rt[e - half].y;
-        }
-        q_full[((size_t)t * H + h) * wide + rank + e] = from_f32<T>(v);
+        q_full[((size_t)t * H + h) * wide + rank + e] = from_f32<T>(turned(row + q_off + h * (dk + dr) + dk, rt, e, rot_dims, pairs));
     }
     // the latent: divided by its root mean square, times its weight
     float sq = 0.0f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) sq = fmaf(row[c_off + i], row[c_off + i], sq);
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) sq = fmaf(crow[c_off + i], crow[c_off + i], sq);
     const float inv = rsqrtf(block_sum(sq, scratch) / (float)rank + eps);
     if (pages == nullptr) return;
     const long long slot = slots[t];
@@ -125,35 +130,26 @@ __global__ void latent_prep_kernel(const float* __restrict__ rows, int ld, int q
     T* dst = pages + (size_t)slot * wide;          // one head: [page][place] is [slot]
     for (int i = threadIdx.x; i < rank; i += blockDim.x) {
         const float w = w_dtype == MM_F32 ? reinterpret_cast<const float*>(norm_w)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(norm_w)[i]);
-        dst[i] = from_f32<T>(row[c_off + i] * inv * w);
+        dst[i] = from_f32<T>(crow[c_off + i] * inv * w);
     }
-    const float* part = row + c_off + rank;
-    for (int e = threadIdx.x; e < dr; e += blockDim.x) {
-        float v = part[e];
-        if (e < half) {
-            v = part[e] * rt[e].x - part[e + half] * rt[e].y;
-        } else if (e < rot_dims) {
-            v = part[e] * rt[e - half].x + part[e - half] * rt[e - half].y;
-        }
-        dst[rank + e] = from_f32<T>(v);
-    }
+    for (int e = threadIdx.x; e < dr; e += blockDim.x) dst[rank + e] = from_f32<T>(turned(crow + c_off + rank, rt, e, rot_dims, pairs));
 }
 
-MM_EXPORT int mm_latent_prep(const void* rows, int ld, int q_off, int c_off, const void* norm_w, int w_dtype, float eps, const void* rot,
-                             int rot_dims, void* q_plain, void* q_full, void* pages, int dtype, const void* slots, int page_size, int n_tokens,
+MM_EXPORT int mm_latent_prep(const void* q_rows, int ldq, int q_off, const void* c_rows, int ldc, int c_off, const void* norm_w, int w_dtype,
+                             float eps, const void* rot, int rot_dims, int pairs, void* q_plain, void* q_full, void* pages, int dtype, const void* slots, int page_size, int n_tokens,
                              int H, int dk, int dr, int rank, void* stream) {
     MM_REQUIRE(n_tokens >= 0 && H > 0 && dk > 0 && dr >= 0 && rank > 0, "latent prep: bad sizes");
     MM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dr && (rot_dims == 0 || rot != nullptr), "latent prep: the rotated dimensions are even and at most the rotated part");
-    MM_REQUIRE(q_off >= 0 && c_off >= 0 && ld >= q_off + H * (dk + dr) && ld >= c_off + rank + dr, "latent prep: the rows are narrower than what is cut out of them");
+    MM_REQUIRE(q_off >= 0 && c_off >= 0 && ldq >= q_off + H * (dk + dr) && ldc >= c_off + rank + dr, "latent prep: the rows are narrower than what is cut out of them");
     MM_REQUIRE(pages == nullptr || (slots != nullptr && page_size > 0), "latent prep: bad page geometry");
     if (n_tokens == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == MM_F32)
-        mm_launch(latent_prep_kernel<float>, dim3(n_tokens), dim3(256), 0, s, (const float*)rows, ld, q_off, c_off, norm_w, w_dtype, eps,
-                  (const float2*)rot, rot_dims, (float*)q_plain, (float*)q_full, (float*)pages, (const int32_t*)slots, page_size, H, dk, dr, rank);
+        mm_launch(latent_prep_kernel<float>, dim3(n_tokens), dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
+                  norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (float*)q_plain, (float*)q_full, (float*)pages, (const int32_t*)slots, page_size, H, dk, dr, rank);
     else if (dtype == MM_BF16)
-        mm_launch(latent_prep_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, s, (const float*)rows, ld, q_off, c_off, norm_w, w_dtype, eps,
-                  (const float2*)rot, rot_dims, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_full, (__nv_bfloat16*)pages, (const int32_t*)slots,
+        mm_launch(latent_prep_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
+                  norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_full, (__nv_bfloat16*)pages, (const int32_t*)slots,
                   page_size, H, dk, dr, rank);
     else
         MM_REQUIRE(false, "latent prep: dtype must be float32 or bfloat16");

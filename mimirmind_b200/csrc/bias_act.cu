@@ -4,21 +4,11 @@
 //   gelu_tanh  0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 //   silu       z / (1 + exp(-z))
 //   relu       max(z, 0)
+//   gelu_erf   0.5 z (1 + erf(z / sqrt(2)))
 #include "common.cuh"
 
-#define ACT_RELU2 0
-#define ACT_GELU_TANH 1
-#define ACT_SILU 2
-#define ACT_RELU 3
-
-__device__ __forceinline__ float apply_act(float z, int act) {
-    switch (act) {
-        case ACT_RELU2: { const float r = fmaxf(z, 0.0f); return r * r; }
-        case ACT_GELU_TANH: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-        case ACT_SILU: return z / (1.0f + expf(-z));
-        default: return fmaxf(z, 0.0f);
-    }
-}
+// act counts from 0 here (squared relu), unary_act's numbers from 1
+__device__ __forceinline__ float apply_act(float z, int act) { return unary_act<false>(z, act + 1); }
 
 template <typename T, typename BT>
 __global__ void bias_act_kernel(const T* __restrict__ x, const BT* __restrict__ bias, T* __restrict__ out, long long total,
@@ -56,7 +46,7 @@ __global__ void bias_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ x, cons
 }
 
 MM_EXPORT int mm_bias_act(const void* x, const void* bias, int bias_dtype, void* out, int dtype, int n, int f, int act, void* stream) {
-    MM_REQUIRE(n >= 0 && f > 0 && act >= 0 && act <= 3, "bias_act: bad sizes or activation");
+    MM_REQUIRE(n >= 0 && f > 0 && act >= 0 && act < MM_ACT_COUNT, "bias_act: bad sizes or activation");
     if (n == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const long long total = (long long)n * f;

@@ -67,10 +67,28 @@ __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { retu
 // ---- gated activations of a two-matrix feed-forward ---------------------------------------------------------------------
 // g, u: the gate's and the up projection's values, both multiplied by `s` first (a weight on the input of the layer
 // passes through both products).  act 0: silu(g) u.  act 1, the clamped form: g <- min(g, limit), u <- clamp(u, -limit,
-// limit), g sigmoid(1.702 g) (u + 1).  FAST: __expf.
+// limit), g sigmoid(1.702 g) (u + 1).  act 2: gelu(g) u with the tanh form of gelu.  FAST: __expf.
 #define MM_GLU_SILU 0
 #define MM_GLU_CLAMPED 1
+#define MM_GLU_GELU_TANH 2
 #define MM_GLU_CLAMPED_ALPHA 1.702f
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+
+// ---- activations of one value: 0 none, 1 squared relu, 2 gelu (tanh form), 3 silu, 4 relu, 5 gelu (exact form) ----------
+#define MM_ACT_COUNT 5
+template <bool FAST>
+__device__ __forceinline__ float unary_act(float z, int act) {
+    switch (act) {
+        case 0: return z;
+        case 1: { const float r = fmaxf(z, 0.0f); return r * r; }
+        case 2: return gelu_tanh(z);
+        case 3: return z / (1.0f + (FAST ? __expf(-z) : expf(-z)));
+        case 5: return gelu_erf(z);
+        default: return fmaxf(z, 0.0f);
+    }
+}
+
 template <bool FAST>
 __device__ __forceinline__ float glu_act(float g, float u, int act, float limit, float s) {
     g *= s;
@@ -81,6 +99,7 @@ __device__ __forceinline__ float glu_act(float g, float u, int act, float limit,
         const float e = FAST ? __expf(-MM_GLU_CLAMPED_ALPHA * g) : expf(-MM_GLU_CLAMPED_ALPHA * g);
         return g / (1.0f + e) * (u + 1.0f);
     }
+    if (act == MM_GLU_GELU_TANH) return gelu_tanh(g) * u;
     const float e = FAST ? __expf(-g) : expf(-g);
     return g / (1.0f + e) * u;
 }

@@ -48,6 +48,7 @@ struct SkinnyArgs {
     void* out;                  // PLAIN [M, ldo] bf16/fp32; SWIGLU [M, ldo] (N/2 columns)
     const void* bias;           // [N] or null (PLAIN, ROPE)
     int bias_dtype, out_dtype;
+    int act;                    // PLAIN: activation after the bias (unary_act's numbers); SWIGLU: the gated activation (glu_act's)
     int M, N, K, ldo;
     int S;                      // K splits = cluster size
     int stages;                 // depth of the TMA ring
@@ -294,6 +295,10 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
 #pragma unroll
                     for (int i = 0; i < 16; ++i) v[i] += sk_w(a.bias, a.bias_dtype, n0 + i);
                 }
+                if (a.act) {
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) v[i] = unary_act<false>(v[i], a.act);
+                }
                 if (a.out_dtype == MM_F32) {
                     float* o = (float*)a.out + (size_t)m * a.ldo + n0;
 #pragma unroll
@@ -306,7 +311,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
             } else if constexpr (EPI == SK_SWIGLU) {
                 float act[8];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) act[i] = v[i] / (1.0f + expf(-v[i])) * v[8 + i];
+                for (int i = 0; i < 8; ++i) act[i] = glu_act<false>(v[i], v[8 + i], a.act, 0.0f, 1.0f);
                 if (a.out_dtype == MM_F32) {
                     float* o = (float*)a.out + (size_t)m * a.ldo + n0 / 2;
                     *reinterpret_cast<float4*>(o) = make_float4(act[0], act[1], act[2], act[3]);
@@ -527,6 +532,22 @@ MM_EXPORT int mm_gemm_skinny(const void* W, const void* x, const void* bias, int
     a.out = out; a.out_dtype = out_dtype; a.ldo = ldo; a.bias = bias; a.bias_dtype = bias_dtype;
     cudaStream_t s = (cudaStream_t)stream;
     return swiglu ? sk_dispatch<SK_SWIGLU>(W, x, ldx, a, s) : sk_dispatch<SK_PLAIN>(W, x, ldx, a, s);
+}
+
+// The same with an activation: gated != 0: another gated one than silu(g) u (glu_act's kinds without a limit); else
+// unary_act's numbers, after the bias.
+MM_EXPORT int mm_gemm_skinny_act(const void* W, const void* x, const void* bias, int bias_dtype, void* out, int out_dtype, int M, int N, int K,
+                                 int ldx, int ldo, int splits, int gated, int act, void* err, void* stream) {
+    SkinnyArgs a;
+    const int rc = sk_common(a, W, x, M, N, K, ldx, splits, nullptr, 0, 0, 0, 0.0f, err);
+    if (rc != MM_OK) return rc;
+    MM_REQUIRE(out_dtype == MM_F32 || out_dtype == MM_BF16, "gemm_skinny: out dtype must be float32 or bfloat16");
+    MM_REQUIRE(gated ? (bias == nullptr && (act == MM_GLU_SILU || act == MM_GLU_GELU_TANH)) : (act >= 0 && act <= MM_ACT_COUNT),
+               "gemm_skinny: unknown activation");
+    MM_REQUIRE(ldo >= (gated ? N / 2 : N) && ldo % 8 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0, "gemm_skinny: output rows must be 16-byte aligned");
+    a.out = out; a.out_dtype = out_dtype; a.ldo = ldo; a.bias = bias; a.bias_dtype = bias_dtype; a.act = act;
+    cudaStream_t s = (cudaStream_t)stream;
+    return gated ? sk_dispatch<SK_SWIGLU>(W, x, ldx, a, s) : sk_dispatch<SK_PLAIN>(W, x, ldx, a, s);
 }
 
 // residual[M, N] (fp32) += x * W^T.  With norm_w: also xw_out[M, N] = bf16(residual * norm_w) and

@@ -69,16 +69,6 @@ struct SharedCtl {
 
 // The epilogue of one warp for its 32 rows (TMEM lanes) of a 128 x 256 accumulator at `taddr`: rows m0 + 32 q + lane,
 // columns n0 .. n0 + 255 of the product.
-// activations a bf16 epilogue may apply after the bias (fp32): 1 squared relu, 2 gelu (tanh form), 3 silu, 4 relu
-__device__ __forceinline__ float epilogue_activation(float z, int act) {
-    switch (act) {
-        case 1: { const float r = fmaxf(z, 0.0f); return r * r; }
-        case 2: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-        case 3: return z / (1.0f + __expf(-z));
-        default: return fmaxf(z, 0.0f);
-    }
-}
-
 template <int EPI>
 __device__ __forceinline__ void epilogue_rows(uint32_t taddr, int m0, int n0, int q, int lane, unsigned char* wstage,
                                               void* __restrict__ out, const void* __restrict__ bias, int bias_dtype, int M,
@@ -130,7 +120,7 @@ __device__ __forceinline__ void epilogue_rows(uint32_t taddr, int m0, int n0, in
                     }
                     if (act != 0) {
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) v[i] = epilogue_activation(v[i], act);
+                        for (int i = 0; i < 32; ++i) v[i] = unary_act<true>(v[i], act);
                     }
 #pragma unroll
                     for (int i = 0; i < 4; ++i)
@@ -516,11 +506,12 @@ int launch_grouped(const CUtensorMap& a, const CUtensorMap& b, void* out, int M,
 // matrices one after the other; tile i of the device-made list `group_tiles` (3 ints each: first row, end row, group; at
 // most 128 rows, never across a group's border; `n_group_tiles` of them, at most `max_group_tiles`) is multiplied with
 // its group's matrix.  out [M, ldo]: bf16 [M, N], or with the SwiGLU epilogue bf16 [M, N/2].
-// glu, limit: another gated activation than silu(g) u in the SwiGLU epilogue (glu_act's kinds in common.cuh).
+// glu, limit: another gated activation than silu(g) u in the SwiGLU epilogue (glu_act's kinds in common.cuh); with the bf16
+// epilogue `glu` is the activation of the product itself (unary_act's numbers).
 MM_EXPORT int mm_gemm_tcgen05_grouped_act(const void* A, const void* W, void* out, int epilogue, int M, int groups, int N, int K, int lda, int ldo,
                                           const void* group_tiles, const void* n_group_tiles, int max_group_tiles, int glu, float limit, void* err,
                                           void* stream) {
-    MM_REQUIRE(glu == 0 || (epilogue == EPI_SWIGLU && glu == MM_GLU_CLAMPED), "gemm_tcgen05 grouped: the gated activations are silu and the clamped form, in the SwiGLU epilogue");
+    MM_REQUIRE(glu >= 0 && glu <= (epilogue == EPI_SWIGLU ? MM_GLU_GELU_TANH : MM_ACT_COUNT), "gemm_tcgen05 grouped: unknown activation");
     MM_REQUIRE(M > 0 && N > 0 && K > 0 && groups > 0 && max_group_tiles > 0 && group_tiles && n_group_tiles, "gemm_tcgen05 grouped: bad sizes");
     MM_REQUIRE(K % 8 == 0 && lda % 8 == 0 && lda >= K, "gemm_tcgen05: K and the row stride of A must be multiples of 8 (16-byte TMA rows)");
     MM_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0 && ((uintptr_t)out & 15) == 0, "gemm_tcgen05: pointers must be 16-byte aligned");
@@ -540,7 +531,7 @@ MM_EXPORT int mm_gemm_tcgen05_grouped_act(const void* A, const void* W, void* ou
         return launch_grouped<EPI_SWIGLU>(ta, tb, out, M, N, K, ldo, (int*)err, sms, (const int32_t*)group_tiles, (const int32_t*)n_group_tiles,
                                           max_group_tiles, N, s, glu, limit);
     return launch_grouped<EPI_BF16>(ta, tb, out, M, N, K, ldo, (int*)err, sms, (const int32_t*)group_tiles, (const int32_t*)n_group_tiles,
-                                    max_group_tiles, N, s);
+                                    max_group_tiles, N, s, glu, 0.0f);
 }
 
 MM_EXPORT int mm_gemm_tcgen05_grouped(const void* A, const void* W, void* out, int epilogue, int M, int groups, int N, int K, int lda, int ldo,
@@ -582,12 +573,18 @@ MM_EXPORT int mm_gemm_tcgen05(const void* A, const void* W, const void* bias, in
     return gemm_tcgen05_common(A, W, bias, bias_dtype, out, epilogue, M, N, K, lda, ldo, err, stream, false);
 }
 
-// out = act(A W^T + bias) as bf16: the plain product with an activation in its epilogue (act: 1 squared relu, 2 gelu in
-// its tanh form, 3 silu, 4 relu), on CTA pairs when `pair` is set.  The hidden rows of a two-matrix feed-forward are made
+// out [M, N/2] = the gated activation `glu` (glu_act's kinds without a limit) of W rows that interleave gate and up in blocks of 8
+MM_EXPORT int mm_gemm_tcgen05_glu(const void* A, const void* W, void* out, int glu, int pair, int M, int N, int K, int lda, int ldo, void* err,
+                                  void* stream) {
+    MM_REQUIRE(glu == MM_GLU_SILU || glu == MM_GLU_GELU_TANH, "gemm_tcgen05: unknown gated activation");
+    return gemm_tcgen05_common(A, W, nullptr, MM_F32 | (glu << 8), out, EPI_SWIGLU, M, N, K, lda, ldo, err, stream, pair != 0);
+}
+
+// out = act(A W^T + bias) as bf16: the plain product with an activation in its epilogue (unary_act's numbers), on CTA pairs when `pair` is set.  The hidden rows of a two-matrix feed-forward are made
 // in one launch and never exist without their activation.
 MM_EXPORT int mm_gemm_tcgen05_act(const void* A, const void* W, const void* bias, int bias_dtype, void* out, int act, int pair, int M,
                                   int N, int K, int lda, int ldo, void* err, void* stream) {
-    MM_REQUIRE(act >= 1 && act <= 4 && (bias_dtype == MM_F32 || bias_dtype == MM_BF16), "gemm_tcgen05: unknown activation or bias dtype");
+    MM_REQUIRE(act >= 1 && act <= MM_ACT_COUNT && (bias_dtype == MM_F32 || bias_dtype == MM_BF16), "gemm_tcgen05: unknown activation or bias dtype");
     return gemm_tcgen05_common(A, W, bias, bias_dtype | (act << 8), out, EPI_BF16, M, N, K, lda, ldo, err, stream, pair != 0);
 }
 

@@ -6,6 +6,9 @@
 //   the `keep` best runs can be chosen; of those the `top` with the largest s are taken (ties: the lower index);
 //   weights: the chosen s divided by their sum (+ 1e-20);
 //   y = sum over the chosen e of weight_e * W_down[e] (act(W_gate[e] x) * (W_up[e] x)).
+// Options: logistic scores that are not renormed; a correction per expert added to the scores for the choice only; runs
+// scored by the sum of their two best choice scores; experts of two matrices, W_down[e] act(W_up[e] x); one more row of the
+// router's matrix whose logistic value gates something else per token.
 //
 // Nothing here waits for the host: the lists are made on the device (route -> sort), the products run over a grid
 // that is large enough for any split of the step's rows between experts (CTAs without a tile return), and the sum
@@ -28,10 +31,17 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {      // the larg
     }
 }
 
-// One warp: the choice for one token from its E logits `zr`; s, gs: the warp's scratch (E and `groups` floats).
+// One warp: the choice for one token from its E logits `zr`; scratch: 2 E + 2 groups floats of the warp's own.
 // scoring 0: s = softmax(z), the chosen weights divided by their sum; 1: s = sigmoid(z), the chosen weights as they are.
-__device__ __forceinline__ void moe_route_warp(const float* zr, float* s, float* gs, int lane, int E, int top, int groups, int keep,
-                                               int32_t* __restrict__ idx, float* __restrict__ wts, size_t t, int scoring = 0) {
+// The choice goes by c = s + correction (null: c = s), which may be negative; a run of experts is scored by its best c, or
+// with pair_sum by the sum of its two best (a run of one: its only one).
+__device__ __forceinline__ void moe_route_warp(const float* zr, float* scratch, int lane, int E, int top, int groups, int keep,
+                                               int32_t* __restrict__ idx, float* __restrict__ wts, size_t t, int scoring = 0,
+                                               const float* __restrict__ correction = nullptr, int pair_sum = 0) {
+    float* s = scratch;
+    float* c = scratch + E;
+    float* gs = scratch + 2 * E;
+    float* kept = gs + groups;
     if (scoring == 1) {
         for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-zr[e]));
     } else {
@@ -48,53 +58,57 @@ __device__ __forceinline__ void moe_route_warp(const float* zr, float* s, float*
         const float inv = 1.0f / sum;
         for (int e = lane; e < E; e += 32) s[e] *= inv;
     }
+    for (int e = lane; e < E; e += 32) c[e] = correction ? s[e] + correction[e] : s[e];
     __syncwarp();
     const int size = E / groups;
     if (keep < groups) {
         for (int g = lane; g < groups; g += 32) {
-            float b = 0.0f;
-            for (int e = 0; e < size; ++e) b = fmaxf(b, s[g * size + e]);
-            gs[g] = b;
+            float b = -INFINITY, b2 = -INFINITY;
+            for (int e = 0; e < size; ++e) {
+                const float v = c[g * size + e];
+                if (v > b) {
+                    b2 = b;
+                    b = v;
+                } else {
+                    b2 = fmaxf(b2, v);
+                }
+            }
+            gs[g] = pair_sum && size > 1 ? b + b2 : b;
         }
         __syncwarp();
-        // the keep best runs get their score replaced by -1: what stays non-negative is dropped
-        for (int kk = 0; kk < keep; ++kk) {
-            float bv = -1.0f;
-            int bi = 0x7fffffff;
-            for (int g = lane; g < groups; g += 32)
-                if (gs[g] >= 0.0f && (gs[g] > bv)) {
-                    bv = gs[g];
-                    bi = g;
-                }
-            warp_argmax(bv, bi);
-            if (lane == 0 && bi != 0x7fffffff) gs[bi] = -1.0f;
-            __syncwarp();
+        // a run stays when fewer than `keep` runs are ahead of it (a better score, or an equal one and a lower index)
+        for (int g = lane; g < groups; g += 32) {
+            int ahead = 0;
+            for (int o = 0; o < groups; ++o) ahead += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+            kept[g] = ahead < keep ? 1.0f : 0.0f;
         }
+        __syncwarp();
         for (int e = lane; e < E; e += 32)
-            if (gs[e / size] >= 0.0f) s[e] = -1.0f - s[e];      // not eligible
+            if (kept[e / size] == 0.0f) c[e] = -INFINITY;      // not eligible
         __syncwarp();
     }
     float total = 0.0f;
     for (int kk = 0; kk < top; ++kk) {
-        float bv = -1.0f;
+        float bv = -INFINITY;
         int bi = 0x7fffffff;
         for (int e = lane; e < E; e += 32)
-            if (s[e] >= 0.0f && s[e] > bv) {
-                bv = s[e];
+            if (c[e] > bv) {
+                bv = c[e];
                 bi = e;
             }
         warp_argmax(bv, bi);
+        float weight = 0.0f;
         if (bi == 0x7fffffff) {     // fewer eligible experts than `top`: the rest of the choice carries no weight
             bi = 0;
-            bv = 0.0f;
-        } else if (lane == 0) {
-            s[bi] = -3.0f;
+        } else {
+            weight = s[bi];
+            if (lane == 0) c[bi] = -INFINITY;
         }
         __syncwarp();
-        total += bv;
+        total += weight;
         if (lane == 0) {
             idx[t * top + kk] = bi;
-            wts[t * top + kk] = bv;
+            wts[t * top + kk] = weight;
         }
     }
     __syncwarp();
@@ -110,8 +124,8 @@ __global__ void moe_route_kernel(const float* __restrict__ z, int ldz, int n_tok
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int t = blockIdx.x * warps + warp;
     if (t >= n_tokens) return;
-    float* s = route_smem + (size_t)warp * (E + groups);
-    moe_route_warp(z + (size_t)t * ldz, s, s + E, lane, E, top, groups, keep, idx, wts, (size_t)t, scoring);
+    float* s = route_smem + (size_t)warp * 2 * (E + groups);
+    moe_route_warp(z + (size_t)t * ldz, s, lane, E, top, groups, keep, idx, wts, (size_t)t, scoring);
 }
 
 // The router's product and its choice in one launch, one block per token: every warp takes experts in turn and sums
@@ -137,12 +151,14 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
 
 template <typename T>
 __global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, int D, int E, int top,
-                                                         int groups, int keep, int vec, int32_t* __restrict__ idx, float* __restrict__ wts, int scoring) {
-    extern __shared__ float route_smem[];      // logits [E], scores [E], runs [groups]
+                                                         int groups, int keep, int vec, int32_t* __restrict__ idx, float* __restrict__ wts, int scoring,
+                                                         const float* __restrict__ correction, int pair_sum, float* __restrict__ gate) {
+    extern __shared__ float route_smem[];      // logits [E + 1], then the choice's scratch
+    const int rows = gate ? E + 1 : E;         // with a gate the matrix has one more row, for it
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const size_t t = blockIdx.x;
     const T* xr = x + t * ldx;
-    for (int e = warp; e < E; e += 8) {
+    for (int e = warp; e < rows; e += 8) {
         const float* we = w + (size_t)e * D;
         float acc = 0.0f;
         if (vec) {        // rows that start on 16-byte boundaries: eight numbers per lane and step, several steps in flight
@@ -166,28 +182,36 @@ __global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ x
         if (lane == 0) route_smem[e] = acc;
     }
     __syncthreads();
-    if (warp == 0) moe_route_warp(route_smem, route_smem + E, route_smem + 2 * E, lane, E, top, groups, keep, idx, wts, t, scoring);
+    if (gate && threadIdx.x == 32) gate[t] = 1.0f / (1.0f + expf(-route_smem[E]));
+    if (warp == 0) moe_route_warp(route_smem, route_smem + E + 1, lane, E, top, groups, keep, idx, wts, t, scoring, correction, pair_sum);
 }
 
-MM_EXPORT int mm_moe_router_scored(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,
-                                   int scoring, void* idx, void* wts, void* stream) {
+// w fp32 [E, D], or [E + 1, D] with `gate` (fp32 [n_tokens]), which gets the logistic of the last row's product;
+// correction fp32 [E] or null
+MM_EXPORT int mm_moe_router_choice(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,
+                                   int scoring, const void* correction, int pair_sum, void* gate, void* idx, void* wts, void* stream) {
     MM_REQUIRE(scoring == 0 || scoring == 1, "moe router: the scoring is 0 (softmax, renormed) or 1 (sigmoid, as it is)");
     MM_REQUIRE(n_tokens >= 0 && D > 0 && ldx >= D && E > 0 && top > 0 && top <= E && groups > 0 && E % groups == 0 && keep > 0 && keep <= groups,
                "moe router: experts must split into equal runs, and 0 < top <= experts, 0 < keep <= runs");
-    MM_REQUIRE((size_t)(2 * E + groups) * sizeof(float) <= 48 * 1024, "moe router: too many experts for the router's shared memory");
+    const size_t smem = (size_t)(3 * E + 1 + 2 * groups) * sizeof(float);
+    MM_REQUIRE(smem <= 48 * 1024, "moe router: too many experts for the router's shared memory");
     if (n_tokens == 0) return MM_OK;
-    const size_t smem = (size_t)(2 * E + groups) * sizeof(float);
     const int vec = D % 8 == 0 && ldx % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
     if (x_dtype == MM_F32)
         mm_launch(moe_router_kernel<float>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, (const float*)x, ldx, (const float*)w, D, E, top,
-                  groups, keep, vec, (int32_t*)idx, (float*)wts, scoring);
+                  groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate);
     else if (x_dtype == MM_BF16)
         mm_launch(moe_router_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, (const __nv_bfloat16*)x, ldx,
-                  (const float*)w, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring);
+                  (const float*)w, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate);
     else
         MM_REQUIRE(false, "moe router: dtype must be float32 or bfloat16");
     MM_CHECK_LAUNCH();
     return MM_OK;
+}
+
+MM_EXPORT int mm_moe_router_scored(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,
+                                   int scoring, void* idx, void* wts, void* stream) {
+    return mm_moe_router_choice(x, x_dtype, ldx, w, n_tokens, D, E, top, groups, keep, scoring, nullptr, 0, nullptr, idx, wts, stream);
 }
 
 MM_EXPORT int mm_moe_router(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,
@@ -198,10 +222,10 @@ MM_EXPORT int mm_moe_router(const void* x, int x_dtype, int ldx, const void* w, 
 MM_EXPORT int mm_moe_route(const void* z, int ldz, int n_tokens, int E, int top, int groups, int keep, void* idx, void* wts, void* stream) {
     MM_REQUIRE(n_tokens >= 0 && E > 0 && top > 0 && top <= E && groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && ldz >= E,
                "moe route: experts must split into equal runs, and 0 < top <= experts, 0 < keep <= runs");
-    MM_REQUIRE((size_t)(E + groups) * 4 * sizeof(float) <= 48 * 1024, "moe route: too many experts for the router's shared memory");
+    MM_REQUIRE((size_t)(E + groups) * 8 * sizeof(float) <= 48 * 1024, "moe route: too many experts for the router's shared memory");
     if (n_tokens == 0) return MM_OK;
     const int warps = 4;
-    mm_launch(moe_route_kernel, dim3(ceil_div(n_tokens, warps)), dim3(warps * 32), (size_t)warps * (E + groups) * sizeof(float),
+    mm_launch(moe_route_kernel, dim3(ceil_div(n_tokens, warps)), dim3(warps * 32), (size_t)warps * 2 * (E + groups) * sizeof(float),
               (cudaStream_t)stream, (const float*)z, ldz, n_tokens, E, top, groups, keep, (int32_t*)idx, (float*)wts, 0);
     MM_CHECK_LAUNCH();
     return MM_OK;
@@ -353,13 +377,17 @@ __device__ __forceinline__ bool moe_tile(const int32_t* __restrict__ offsets, in
 #define MOE_MMA_BK 64
 #define MOE_STAGES 3
 
-// fp32 FMA units, every output summed over k in ascending order.  GATED: W is [E, 2F, K], the gate's rows then the
-// up rows, and the output is act(gate) * up over F columns, the input rows gathered through order / top; otherwise
-// W is [E, N, K], the input rows are the sorted ones and output row order[i] is written.
-template <typename TA, typename TW, typename TC, bool GATED>
+// What a product of the experts reads and writes.  GATED: W is [E, 2F, K], the gate's rows then the up rows, and the output
+// is act(gate) * up over F columns, the input rows gathered through order / top; SINGLE: W is [E, F, K], the output act(up), the input
+// rows gathered likewise; DOWN: W is [E, N, K], the input rows are the sorted ones and output row order[i] is written.
+enum { MOE_DOWN = 0, MOE_GATED = 1, MOE_SINGLE = 2 };
+
+// fp32 FMA units, every output summed over k in ascending order.
+template <typename TA, typename TW, typename TC, int MODE>
 __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W, TC* __restrict__ C, int ldc,
                                                             const int32_t* __restrict__ offsets, const int32_t* __restrict__ order, int E, int top,
                                                             int N, int K, int act, float limit, const float* __restrict__ row_scale) {
+    constexpr bool GATED = MODE == MOE_GATED, GATHER = MODE != MOE_DOWN;
     __shared__ float As[MOE_BK][MOE_BM + 4];
     __shared__ float Ws[MOE_BK][MOE_BN + 4];
     __shared__ float Us[GATED ? MOE_BK : 1][MOE_BN + 4];
@@ -377,7 +405,7 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const TA* __restrict
     const int e = tile_info[0], lo = tile_info[1], hi = tile_info[2];
     if (e < 0) return;
     const int M = hi - lo;
-    if (tid < MOE_BM) rows[tid] = tid < M ? (GATED ? order[lo + tid] / top : lo + tid) : 0;
+    if (tid < MOE_BM) rows[tid] = tid < M ? (GATHER ? order[lo + tid] / top : lo + tid) : 0;
     __syncthreads();
     const int tx = tid & 15, ty = tid >> 4;
     const int n0 = blockIdx.x * MOE_BN;
@@ -433,13 +461,14 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const TA* __restrict
     for (int i = 0; i < 4; ++i) {
         const int m = ty * 4 + i;
         if (m >= M) continue;
-        const size_t out_row = GATED ? (size_t)(lo + m) : (size_t)order[lo + m];
+        const size_t out_row = GATHER ? (size_t)(lo + m) : (size_t)order[lo + m];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
             if (GATED) v = glu_act<false>(v, up[i][j], act, limit, row_scale ? row_scale[order[lo + m]] : 1.0f);
+            if (MODE == MOE_SINGLE) v = unary_act<false>(row_scale ? v * row_scale[order[lo + m]] : v, act);
             C[out_row * ldc + n] = from_f32<TC>(v);
         }
     }
@@ -447,7 +476,7 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const TA* __restrict
 
 // bfloat16 on the tensor cores (mma.sync m16n8k16, fp32 accumulation): the same tiles, 64 rows x 64 columns, four
 // warps of 32 x 32 (gated: gate and up accumulators side by side), K in steps of 64 through a ring of shared-memory stages.
-template <bool GATED, typename TC>
+template <int MODE, typename TC>
 __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W,
                                                            TC* __restrict__ C, int ldc, const int32_t* __restrict__ offsets,
                                                            const int32_t* __restrict__ order, int E, int top, int N, int K, int interleaved, int act, float limit,
@@ -455,6 +484,7 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
     // K in steps of 64 through a ring of MOE_STAGES stages: a decode step's tiles hold a handful of rows and stream a
     // whole expert, so what counts is how many bytes of weights a CTA keeps in flight (rows of 144 bytes: ldmatrix
     // reads without bank conflicts)
+    constexpr bool GATED = MODE == MOE_GATED, GATHER = MODE != MOE_DOWN;
     constexpr int BK = MOE_MMA_BK, LD = BK + 8;
     constexpr int WROWS_ = GATED ? 2 * MOE_BN : MOE_BN;
     extern __shared__ __align__(16) unsigned char moe_smem[];
@@ -476,7 +506,7 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
     const int e = tile_info[0], lo = tile_info[1], hi = tile_info[2];
     if (e < 0) return;
     const int M = hi - lo;
-    if (tid < MOE_BM) rows[tid] = tid < M ? (GATED ? order[lo + tid] / top : lo + tid) : -1;
+    if (tid < MOE_BM) rows[tid] = tid < M ? (GATHER ? order[lo + tid] / top : lo + tid) : -1;
     __syncthreads();
     const int warp = tid >> 5, lane = tid & 31;
     const int wm = (warp >> 1) * 32, wn = (warp & 1) * 32;
@@ -559,7 +589,7 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
         for (int half = 0; half < 2; ++half) {
             const int m = wm + mi * 16 + (lane >> 2) + half * 8;
             if (m >= M) continue;
-            const size_t out_row = GATED ? (size_t)(lo + m) : (size_t)order[lo + m];
+            const size_t out_row = GATHER ? (size_t)(lo + m) : (size_t)order[lo + m];
 #pragma unroll
             for (int ni = 0; ni < 4; ++ni)
 #pragma unroll
@@ -568,6 +598,7 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
                     if (n >= N) continue;
                     float v = acc[mi][ni][half * 2 + c];
                     if (GATED) v = glu_act<true>(v, up[mi][ni][half * 2 + c], act, limit, row_scale ? row_scale[order[lo + m]] : 1.0f);
+                    if (MODE == MOE_SINGLE) v = unary_act<true>(row_scale ? v * row_scale[order[lo + m]] : v, act);
                     C[out_row * ldc + n] = from_f32<TC>(v);
                 }
         }
@@ -575,17 +606,17 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
 
 // A [rows, lda] (gated: the step's tokens; else the sorted hidden rows), W the experts' stacked matrices, C: gated
 // [n_rows, N] in sorted order, else [n_rows, N] with row order[i] written.  n_rows = tokens * top.
-// act: what a gated product does with its two halves (glu_act in common.cuh: 0 silu(g) u; 1 the clamped form with
-// `limit`); row_scale [tokens * top] fp32 or null: row (token * top + choice) of a gated product is multiplied by it
+// gated: 0 the plain product, 1 gate and up, 2 one matrix with an activation.  act: what a gated product does with its two
+// halves (glu_act in common.cuh) or a product with one matrix with its result (unary_act); row_scale [tokens * top] fp32 or null: row (token * top + choice) of a gated product is multiplied by it
 // before the activation (a weight on the expert's input: W (s x) = s (W x)).
 MM_EXPORT int mm_moe_gemm_act(const void* A, int a_dtype, int lda, const void* W, int w_dtype, void* C, int c_dtype, int ldc, const void* offsets,
                               const void* order, int n_rows, int E, int top, int N, int K, int gated, int tensor_cores, int interleaved,
                               int act, float limit, const void* row_scale_, void* stream) {
     const float* row_scale = (const float*)row_scale_;
-    MM_REQUIRE(act == 0 || act == 1, "moe gemm: the activation is 0 (silu) or 1 (clamped)");
+    MM_REQUIRE(gated >= 0 && gated <= 2 && act >= 0 && act <= (gated == 2 ? MM_ACT_COUNT : MM_GLU_GELU_TANH), "moe gemm: unknown kind of product or activation");
     MM_REQUIRE(gated || (act == 0 && row_scale == nullptr), "moe gemm: activation and row scale belong to the gated product");
     MM_REQUIRE(n_rows >= 0 && E > 0 && top > 0 && N > 0 && K > 0 && lda >= K && ldc >= N, "moe gemm: bad sizes");
-    MM_REQUIRE(!interleaved || (gated && N % 8 == 0), "moe gemm: interleaved gate and up rows need a gated product of a multiple of 8 columns");
+    MM_REQUIRE(!interleaved || (gated == 1 && N % 8 == 0), "moe gemm: interleaved gate and up rows need a gated product of a multiple of 8 columns");
     if (n_rows == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid(ceil_div(N, MOE_BN), ceil_div(n_rows, MOE_BM) + E);
@@ -593,20 +624,23 @@ MM_EXPORT int mm_moe_gemm_act(const void* A, int a_dtype, int lda, const void* W
     const int32_t* off = (const int32_t*)offsets;
     const int32_t* ord = (const int32_t*)order;
     if (tensor_cores && a_dtype == MM_BF16 && w_dtype == MM_BF16 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
-        const size_t tile_smem = sizeof(bf) * MOE_STAGES * (MOE_BM + (gated ? 2 : 1) * MOE_BN) * (MOE_MMA_BK + 8);
+        const size_t tile_smem = sizeof(bf) * MOE_STAGES * (MOE_BM + (gated == 1 ? 2 : 1) * MOE_BN) * (MOE_MMA_BK + 8);
         static bool configured = false;
         if (!configured) {
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<true, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + 2 * MOE_BN) * (MOE_MMA_BK + 8)));
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<false, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<false, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_GATED, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + 2 * MOE_BN) * (MOE_MMA_BK + 8)));
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_SINGLE, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_DOWN, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_DOWN, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
             configured = true;
         }
-        if (gated && c_dtype == MM_BF16)
-            mm_launch(moe_gemm_mma_kernel<true, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, interleaved, act, limit, row_scale);
+        if (gated == 2 && c_dtype == MM_BF16)
+            mm_launch(moe_gemm_mma_kernel<MOE_SINGLE, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, 0, act, limit, row_scale);
+        else if (gated && c_dtype == MM_BF16)
+            mm_launch(moe_gemm_mma_kernel<MOE_GATED, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, interleaved, act, limit, row_scale);
         else if (!gated && c_dtype == MM_BF16)
-            mm_launch(moe_gemm_mma_kernel<false, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, 0, 0, 0.0f, (const float*)nullptr);
+            mm_launch(moe_gemm_mma_kernel<MOE_DOWN, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, 0, 0, 0.0f, (const float*)nullptr);
         else if (!gated && c_dtype == MM_F32)
-            mm_launch(moe_gemm_mma_kernel<false, float>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (float*)C, ldc, off, ord, E, top, N, K, 0, 0, 0.0f, (const float*)nullptr);
+            mm_launch(moe_gemm_mma_kernel<MOE_DOWN, float>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (float*)C, ldc, off, ord, E, top, N, K, 0, 0, 0.0f, (const float*)nullptr);
         else
             MM_REQUIRE(false, "moe gemm: this combination of dtypes is not built");
         MM_CHECK_LAUNCH();
@@ -615,10 +649,12 @@ MM_EXPORT int mm_moe_gemm_act(const void* A, int a_dtype, int lda, const void* W
     MM_REQUIRE(!interleaved, "moe gemm: interleaved gate and up rows are read by the tensor-core kernels only");
 #define MOE_SIMT(TA, TW, TC)                                                                                                                  \
     do {                                                                                                                                      \
-        if (gated)                                                                                                                            \
-            mm_launch(moe_gemm_simt_kernel<TA, TW, TC, true>, grid, dim3(256), 0, s, (const TA*)A, lda, (const TW*)W, (TC*)C, ldc, off, ord, E, top, N, K, act, limit, row_scale); \
+        if (gated == 2)                                                                                                                       \
+            mm_launch(moe_gemm_simt_kernel<TA, TW, TC, MOE_SINGLE>, grid, dim3(256), 0, s, (const TA*)A, lda, (const TW*)W, (TC*)C, ldc, off, ord, E, top, N, K, act, limit, row_scale); \
+        else if (gated)                                                                                                                       \
+            mm_launch(moe_gemm_simt_kernel<TA, TW, TC, MOE_GATED>, grid, dim3(256), 0, s, (const TA*)A, lda, (const TW*)W, (TC*)C, ldc, off, ord, E, top, N, K, act, limit, row_scale); \
         else                                                                                                                                  \
-            mm_launch(moe_gemm_simt_kernel<TA, TW, TC, false>, grid, dim3(256), 0, s, (const TA*)A, lda, (const TW*)W, (TC*)C, ldc, off, ord, E, top, N, K, 0, 0.0f, (const float*)nullptr); \
+            mm_launch(moe_gemm_simt_kernel<TA, TW, TC, MOE_DOWN>, grid, dim3(256), 0, s, (const TA*)A, lda, (const TW*)W, (TC*)C, ldc, off, ord, E, top, N, K, 0, 0.0f, (const float*)nullptr); \
     } while (0)
     if (a_dtype == MM_F32 && w_dtype == MM_F32 && c_dtype == MM_F32) MOE_SIMT(float, float, float);
     else if (a_dtype == MM_BF16 && w_dtype == MM_BF16 && c_dtype == MM_BF16) MOE_SIMT(bf, bf, bf);

@@ -191,7 +191,7 @@ def _latent_lib():
         P, I, F = c_void_p, c_int, c_float
         _lib.declare("mm_attention_latent_supported", [I, I])
         _lib.declare("mm_attention_latent_tile_rows", [I])
-        _lib.declare("mm_attention_latent_bf16", [P, P, P, P, P, I, P, I, I, I, P, P, I, I, I, I, I, I, F, I, P])
+        _lib.declare("mm_attention_latent_bf16", [P, P, P, P, P, I, P, I, I, I, P, P, I, I, I, I, I, I, F, P, I, P])
         _latent_declared = True
     return _lib.load()
 
@@ -218,9 +218,10 @@ def latent_plan(ctx, num_heads: int, tile_rows: int = LATENT_TILE_ROWS):
     return plan
 
 
-def paged_latent_attention(q, pages, cache, out, ctx, num_heads: int, wide: int, rank: int, window: int, scale: float) -> torch.Tensor:
+def paged_latent_attention(q, pages, cache, out, ctx, num_heads: int, wide: int, rank: int, window: int, scale: float, sink=None) -> torch.Tensor:
     """Attention of ``num_heads`` query heads of ``wide`` numbers over one shared key head ``pages`` [pages, 1, page, wide]
-    whose leading ``rank`` numbers are the value; ``out`` [n, num_heads * rank].  bfloat16 with a rank the tensor-core
+    whose leading ``rank`` numbers are the value, with a learned ``sink`` per head (fp32 [num_heads], or None) in the softmax's
+    denominator; ``out`` [n, num_heads * rank].  bfloat16 with a rank the tensor-core
     kernel is built for: that kernel, its key tiles shared out over several CTAs while the step has few query tiles;
     anything else: the fp32-arithmetic kernel."""
     if USE_LATENT_MMA and q.dtype == torch.bfloat16 and scale > 0 and _latent_lib().mm_attention_latent_supported(wide, rank):
@@ -246,10 +247,10 @@ def paged_latent_attention(q, pages, cache, out, ctx, num_heads: int, wide: int,
                                            part_ml.data_ptr() if part_ml is not None else None, splits, tiles.data_ptr(), n_tiles, tile_rows, n_rows,
                                            ctx.positions.data_ptr(), cache.block_table.data_ptr(), cache.block_table.shape[1],
                                            cache.page_size, num_heads, wide, rank, int(window), float(scale),
-                                           int(out.dtype == torch.float32), ops._stream()), "attention_latent_bf16")
+                                           sink.data_ptr() if sink is not None else None, int(out.dtype == torch.float32), ops._stream()), "attention_latent_bf16")
         return out
     return ops.attention_sink_generic(q, pages, pages, out, ctx.positions, ctx.token_req, cache.block_table, cache.page_size, num_heads,
-                                      1, wide, rank, window, scale, False, value_heads=1, value_row=wide)
+                                      1, wide, rank, window, scale, False, sink_logit=sink, value_heads=1, value_row=wide)
 
 
 TALKING_TARGET_CTAS = 2 * 148    # blocks wanted by a step of few tokens: a token's keys are shared out until the GPU is full

@@ -79,12 +79,13 @@ _PROTOTYPES = {
     "mm_stream_copies": [P, P, I, I, I, P],
     "mm_hc_read": [P, P, P, P, I, F, P, I, I, I, I, P],
     "mm_hc_write": [P, P, I, P, P, P, P, P, I, F, P, I, I, I, I, P],
-    "mm_rope_half_table": [P, P, P, P, I, I, P],
+    "mm_rope_half_table": [P, P, P, P, I, I, F, P],
     "mm_qkv_split_post": [P, I, I, I, I, P, P, P, I, P, I, I, I, I, I, I, I, P],
-    "mm_latent_prep": [P, I, I, I, P, I, F, P, I, P, P, P, I, P, I, I, I, I, I, I, P],
+    "mm_latent_prep": [P, I, I, P, I, I, P, I, F, P, I, I, P, P, P, I, P, I, I, I, I, I, I, P],
     "mm_head_matmul": [P, c_longlong, I, P, P, c_longlong, I, I, I, I, I, I, P],
     "mm_head_finish": [P, I, I, F, I, F, F, P, I, P, I, I, I, I, I, P],
     "mm_moe_router_scored": [P, I, I, P, I, I, I, I, I, I, I, P, P, P],
+    "mm_moe_router_choice": [P, I, I, P, I, I, I, I, I, I, I, P, I, P, P, P, P],
     "mm_moe_gemm_act": [P, I, I, P, I, P, I, I, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
     "mm_gemm_tcgen05_grouped_act": [P, P, P, I, I, I, I, I, I, I, P, P, I, I, F, P, P],
     "mm_moe_gather_scaled": [P, I, P, P, P, P, I, I, P],
@@ -94,9 +95,13 @@ _PROTOTYPES = {
     "mm_forget_gate_walk": [P, P, P, I, I, I, P, P, c_longlong, P, P, P, I, I, I, I, P],
     "mm_forget_gate_chunked": [P, P, P, I, I, I, P, P, c_longlong, P, P, P, P, I, I, I, I, I, P, P, P],
     "mm_post_norm": [P, P, P, I, P, P, I, I, I, F, F, F, F, P],
-    "mm_glu_rows": [P, I, c_longlong, P, I, I, I, I, F, P, P],
+    "mm_output_norm": [P, P, I, P, P, I, P, I, P, P, P, I, I, I, F, F, F, F, P],
+    "mm_gemv_bf16_glu": [P, P, P, I, I, I, I, I, I, I, I, I, P],
+    "mm_gemm_skinny_act": [P, P, P, I, P, I, I, I, I, I, I, I, I, I, P, P],
+    "mm_gemm_tcgen05_glu": [P, P, P, I, I, I, I, I, I, I, P, P],
+    "mm_glu_rows": [P, I, c_longlong, P, I, I, I, I, F, P, I, P],
     "mm_cast_rows": [P, P, I, c_longlong, P],
-    "mm_scaled_sum2": [P, P, P, I, c_longlong, F, F, P],
+    "mm_scaled_sum2": [P, P, P, I, c_longlong, F, F, P, I, P],
     "mm_gemm_tcgen05_grouped": [P, P, P, I, I, I, I, I, I, I, P, P, I, P, P],
 }
 

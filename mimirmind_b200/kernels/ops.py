@@ -845,28 +845,68 @@ def mingru_chunked(a: torch.Tensor, y: torch.Tensor, state: torch.Tensor, chunk_
     return y
 
 
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "relu": 3}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "gelu_erf": 4}
 
 
 def gemv_bf16_act(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], activation: str) -> torch.Tensor:
-    """act(x[M<=8, K] @ w[N, K]^T + bias) in one launch of the weight-streaming kernel (the activation on the fp32 sums)."""
+    """act(x[M<=64, K] @ w[N, K]^T + bias) in one launch of a weight-streaming kernel (the activation on the fp32 sums)."""
     _need(x, "gemv x", torch.bfloat16)
     _need(w, "gemv w", torch.bfloat16)
     m, k = x.shape
     n = w.shape[0]
-    if w.shape != (n, k) or not gemv_supported(m, n, k):
+    if w.shape != (n, k) or not small_batch_supported(m, n, k):
         raise KernelError(f"gemv: shapes x{tuple(x.shape)} w{tuple(w.shape)} are not supported")
     if bias is not None:
         _need(bias, "gemv bias")
     out = torch.empty((m, n), dtype=torch.bfloat16, device=x.device)
+    if m > GEMV_MAX_ROWS:
+        check(_lib.load().mm_gemm_skinny_act(w.data_ptr(), x.data_ptr(), _ptr(bias), dtype_code(bias.dtype) if bias is not None else F32,
+                                             out.data_ptr(), BF16, m, n, k, k, n, _skinny_splits(n, k), 0, ACTIVATIONS[activation] + 1,
+                                             tcgen05_error_flag(x.device).data_ptr(), _stream()), "gemm_skinny_act")
+        return out
     rt, ks = _gemv_layout(n, k)
     check(_lib.load().mm_gemv_bf16_act(w.data_ptr(), x.data_ptr(), _ptr(bias), dtype_code(bias.dtype) if bias is not None else F32,
                                        out.data_ptr(), BF16, m, n, k, k, n, rt, ks, ACTIVATIONS[activation] + 1, _stream()), "gemv_bf16_act")
     return out
 
 
+def gemv_bf16_glu(x: torch.Tensor, w: torch.Tensor, activation: str) -> torch.Tensor:
+    """The gated activation of x[M<=64, K] @ w[2F, K]^T, gate and up rows of ``w`` interleaved in blocks of 8: [M, F] bfloat16 in
+    one launch of a weight-streaming kernel (``activation`` of GLU_ACTIVATIONS, one without a limit)."""
+    _need(x, "gemv x", torch.bfloat16)
+    _need(w, "gemv w", torch.bfloat16)
+    m, k = x.shape
+    n = w.shape[0]
+    if w.shape != (n, k) or not small_batch_supported(m, n, k):
+        raise KernelError(f"gemv: shapes x{tuple(x.shape)} w{tuple(w.shape)} are not supported")
+    out = torch.empty((m, n // 2), dtype=torch.bfloat16, device=x.device)
+    if m > GEMV_MAX_ROWS:
+        check(_lib.load().mm_gemm_skinny_act(w.data_ptr(), x.data_ptr(), None, F32, out.data_ptr(), BF16, m, n, k, k, n // 2, _skinny_splits(n, k), 1,
+                                             GLU_ACTIVATIONS[activation], tcgen05_error_flag(x.device).data_ptr(), _stream()), "gemm_skinny_act")
+        return out
+    rt, ks = _gemv_layout(n, k)
+    check(_lib.load().mm_gemv_bf16_glu(w.data_ptr(), x.data_ptr(), out.data_ptr(), BF16, m, n, k, k, n // 2, rt, ks, GLU_ACTIVATIONS[activation],
+                                       _stream()), "gemv_bf16_glu")
+    return out
+
+
+def gemm_tcgen05_glu(x: torch.Tensor, w: torch.Tensor, activation: str, pair: Optional[bool] = None) -> torch.Tensor:
+    """The same for prompt-sized steps on the tcgen05 tensor cores, the gated activation in the product's epilogue."""
+    _need(x, "gemm x", torch.bfloat16)
+    _need(w, "gemm w", torch.bfloat16)
+    m, k = x.shape
+    n = w.shape[0]
+    if w.shape != (n, k) or n % 16 or not gemm_tcgen05_supported(m, n, k):
+        raise KernelError(f"gemm_tcgen05: shapes x{tuple(x.shape)} w{tuple(w.shape)} are not supported")
+    out = torch.empty((m, n // 2), dtype=torch.bfloat16, device=x.device)
+    check(_lib.load().mm_gemm_tcgen05_glu(x.data_ptr(), w.data_ptr(), out.data_ptr(), GLU_ACTIVATIONS[activation],
+                                          int(tcgen05_pair_suits(m) if pair is None else pair), m, n, k, k, n // 2,
+                                          tcgen05_error_flag(x.device).data_ptr(), _stream()), "gemm_tcgen05_glu")
+    return out
+
+
 def bias_act(x: torch.Tensor, bias: Optional[torch.Tensor], activation: str, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out = act(x + bias) in fp32 arithmetic; ``activation`` one of relu2 (squared relu), gelu_tanh, silu, relu."""
+    """out = act(x + bias) in fp32 arithmetic; ``activation`` one of relu2 (squared relu), gelu_tanh, silu, relu, gelu_erf."""
     _need(x, "bias_act x")
     if activation not in ACTIVATIONS:
         raise KernelError(f"activation '{activation}' is not one of {', '.join(sorted(ACTIVATIONS))}")
@@ -1091,21 +1131,33 @@ def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int):
 ROUTER_SCORINGS = {"softmax": 0, "sigmoid": 1}
 
 
-def moe_router(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: int, scoring: str = "softmax"):
+GROUP_SCORES = {"max": 0, "top2_sum": 1}
+
+
+def moe_router(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: int, scoring: str = "softmax",
+               correction: Optional[torch.Tensor] = None, group_score: str = "max", gate: bool = False):
     """The router's product (fp32 sums over ``x`` [n, D] and the fp32 matrix ``w`` [E, D]) and its choice in one launch:
     (experts int32 [n, top], weights fp32 [n, top]).  ``scoring``: ``softmax`` (the chosen scores divided by their sum) or
-    ``sigmoid`` (the chosen scores as they are)."""
+    ``sigmoid`` (the chosen scores as they are).  ``correction`` fp32 [E] is added to the scores for the choice only;
+    ``group_score``: a run of experts counts by its best choice score, or by the sum of its two best.  With ``gate`` the matrix
+    has one more row, whose product's logistic value comes back as a third result, fp32 [n]."""
     _need(x, "router rows")
     _need(w, "router matrix", torch.float32)
     n, D = x.shape
-    E = w.shape[0]
-    if w.shape[1] != D:
+    E = w.shape[0] - int(gate)
+    if w.shape[1] != D or E < 1:
         raise KernelError("moe router: shape mismatch")
+    if correction is not None:
+        _need(correction, "router correction", torch.float32)
+        if correction.numel() != E:
+            raise KernelError("moe router: one correction per expert")
+    gates = torch.empty((n,), dtype=torch.float32, device=x.device) if gate else None
     idx = torch.empty((n, top), dtype=torch.int32, device=x.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=x.device)
-    check(_lib.load().mm_moe_router_scored(x.data_ptr(), dtype_code(x.dtype), D, w.data_ptr(), n, D, E, int(top), int(groups), int(keep),
-                                           ROUTER_SCORINGS[scoring], idx.data_ptr(), wts.data_ptr(), _stream()), "moe_router")
-    return idx, wts
+    check(_lib.load().mm_moe_router_choice(x.data_ptr(), dtype_code(x.dtype), D, w.data_ptr(), n, D, E, int(top), int(groups), int(keep),
+                                           ROUTER_SCORINGS[scoring], _ptr(correction), GROUP_SCORES[group_score], _ptr(gates), idx.data_ptr(),
+                                           wts.data_ptr(), _stream()), "moe_router")
+    return (idx, wts, gates) if gate else (idx, wts)
 
 
 MOE_TILE_ROWS = 128       # rows of a tile of the grouped tensor-memory product
@@ -1144,18 +1196,19 @@ def moe_sort(idx: torch.Tensor, experts: int, with_tiles: bool = False) -> Exper
     return out
 
 
-GLU_ACTIVATIONS = {"silu": 0, "clamped": 1}
+GLU_ACTIVATIONS = {"silu": 0, "clamped": 1, "gelu_tanh": 2}
 
 
 def moe_gemm(a: torch.Tensor, w: torch.Tensor, rows: ExpertRows, n_rows: int, top: int, gated: bool,
              out_dtype: torch.dtype, tensor_cores: bool = True, interleaved: bool = False, activation: str = "silu", limit: float = 0.0,
-             row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+             row_scale: Optional[torch.Tensor] = None, single: bool = False) -> torch.Tensor:
     """The experts' products over their rows.  ``gated``: ``a`` [tokens, K] are the step's rows, ``w`` [E, 2F, K] the gate's
     rows then the up rows of every expert (``interleaved``: alternating in blocks of 8), result ``silu(gate) * up``
     [n_rows, F] in sorted order.  Otherwise ``a`` [n_rows, K] are sorted rows, ``w`` [E, N, K], and row ``order[i]`` of the
     result [n_rows, N] gets sorted row i's product.  A gated product may take another ``activation`` (``clamped``:
     ``g = min(g, limit)``, ``u = clamp(u, -limit, limit)``, ``g sigmoid(1.702 g) (u + 1)``) and a ``row_scale`` fp32 [tokens, top]
-    that multiplies both halves of a (token, choice) row before it (a weight on the expert's input)."""
+    that multiplies both halves of a (token, choice) row before it (a weight on the expert's input).  ``single``: like a gated
+    product, but the experts have one first matrix, ``w`` [E, F, K], and the result is ``activation`` (of ACTIVATIONS) of it."""
     _need(a, "moe rows")
     if row_scale is not None:
         _need(row_scale, "moe row scale", torch.float32)
@@ -1164,12 +1217,15 @@ def moe_gemm(a: torch.Tensor, w: torch.Tensor, rows: ExpertRows, n_rows: int, to
     _need(w, "moe weights", a.dtype)
     E, rows_w, K = w.shape
     N = rows_w // 2 if gated else rows_w
-    if a.shape[1] != K or (not gated and a.shape[0] != n_rows):
+    if single and (gated or interleaved):
+        raise KernelError("moe gemm: a product is gated or has one matrix")
+    if a.shape[1] != K or (not (gated or single) and a.shape[0] != n_rows):
         raise KernelError("moe gemm: shape mismatch")
     out = torch.empty((n_rows, N), dtype=out_dtype, device=a.device)
     check(_lib.load().mm_moe_gemm_act(a.data_ptr(), dtype_code(a.dtype), a.stride(0), w.data_ptr(), dtype_code(w.dtype), out.data_ptr(),
                                       dtype_code(out_dtype), N, rows.offsets.data_ptr(), rows.order.data_ptr(), int(n_rows), E, int(top), N, K,
-                                      int(bool(gated)), int(bool(tensor_cores)), int(bool(interleaved)), GLU_ACTIVATIONS[activation],
+                                      2 if single else int(bool(gated)), int(bool(tensor_cores)), int(bool(interleaved)),
+                                      ACTIVATIONS[activation] + 1 if single else (GLU_ACTIVATIONS[activation] if gated else 0),
                                       float(limit), _ptr(row_scale), _stream()), "moe_gemm")
     return out
 
@@ -1189,10 +1245,12 @@ def moe_gather_scaled(x: torch.Tensor, rows: ExpertRows, wts: Optional[torch.Ten
     return out
 
 
-def moe_gemm_grouped(a: torch.Tensor, w: torch.Tensor, rows: ExpertRows, swiglu: bool, activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
+def moe_gemm_grouped(a: torch.Tensor, w: torch.Tensor, rows: ExpertRows, swiglu: bool, activation: Optional[str] = "silu", limit: float = 0.0,
+                     single: bool = False) -> torch.Tensor:
     """The grouped tensor-memory product: ``a`` [n_rows, K] bf16 in sorted order, ``w`` [E, N, K] bf16; every row tile of
     ``rows.tiles`` times its expert's matrix.  ``swiglu``: the matrix interleaves gate and up rows in blocks of 8 and the
-    result is ``silu(gate) * up`` [n_rows, N/2]; else [n_rows, N].  bf16, in sorted order."""
+    result is ``silu(gate) * up`` [n_rows, N/2] (or another gated ``activation``); else [n_rows, N], with ``single`` after ``activation``
+    (of ACTIVATIONS).  bf16, in sorted order."""
     _need(a, "moe rows", torch.bfloat16)
     _need(w, "moe weights", torch.bfloat16)
     if rows.tiles is None:
@@ -1202,7 +1260,7 @@ def moe_gemm_grouped(a: torch.Tensor, w: torch.Tensor, rows: ExpertRows, swiglu:
     out = torch.empty((n_rows, N // 2 if swiglu else N), dtype=torch.bfloat16, device=a.device)
     check(_lib.load().mm_gemm_tcgen05_grouped_act(a.data_ptr(), w.data_ptr(), out.data_ptr(), 1 if swiglu else 0, n_rows, E, N, K, K, out.shape[1],
                                                   rows.tiles.data_ptr(), rows.n_tiles.data_ptr(), rows.max_tiles,
-                                                  GLU_ACTIVATIONS[activation] if swiglu else 0, float(limit),
+                                                  GLU_ACTIVATIONS[activation] if swiglu else (ACTIVATIONS[activation] + 1 if single else 0), float(limit),
                                                   tcgen05_error_flag(a.device).data_ptr(), _stream()), "gemm_tcgen05_grouped")
     return out
 
@@ -1293,8 +1351,8 @@ def hc_write(x: torch.Tensor, streams: int, y: torch.Tensor, scale: Optional[tor
 
 
 # ---- steps around an attention kernel (csrc/attention_parts.cu) --------------------------------------------------------
-def rope_half_table(positions: torch.Tensor, f_hi: torch.Tensor, f_lo: torch.Tensor) -> torch.Tensor:
-    """(cos, sin) of ``position * (f_hi[i] + f_lo[i])`` as fp32 [n, len(f_hi), 2]; the two words of each frequency come from
+def rope_half_table(positions: torch.Tensor, f_hi: torch.Tensor, f_lo: torch.Tensor, factor: float = 1.0) -> torch.Tensor:
+    """(cos, sin) of ``position * (f_hi[i] + f_lo[i])``, both times ``factor``, as fp32 [n, len(f_hi), 2]; the two words of each frequency come from
     its float64 value, and the rounding of the product is carried, so the angle is good to the last bit of an fp32."""
     _need(positions, "positions", torch.int32)
     _need(f_hi, "frequencies", torch.float32)
@@ -1303,7 +1361,8 @@ def rope_half_table(positions: torch.Tensor, f_hi: torch.Tensor, f_lo: torch.Ten
     if f_lo.numel() != half or half < 1:
         raise KernelError("rotation table: bad sizes")
     out = torch.empty((n, half, 2), dtype=torch.float32, device=positions.device)
-    check(_lib.load().mm_rope_half_table(positions.data_ptr(), f_hi.data_ptr(), f_lo.data_ptr(), out.data_ptr(), n, half, _stream()), "rope_half_table")
+    check(_lib.load().mm_rope_half_table(positions.data_ptr(), f_hi.data_ptr(), f_lo.data_ptr(), out.data_ptr(), n, half, float(factor), _stream()),
+          "rope_half_table")
     return out
 
 
@@ -1332,15 +1391,18 @@ def qkv_split_post(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out
 
 def latent_prep(rows: torch.Tensor, q_off: int, c_off: int, norm_weight: torch.Tensor, eps: float, rot: Optional[torch.Tensor], rot_dims: int,
                 q_plain: torch.Tensor, q_full: torch.Tensor, pages: Optional[torch.Tensor], slots: Optional[torch.Tensor], page_size: int,
-                heads: int, dim: int, rot_dim: int, rank: int) -> None:
+                heads: int, dim: int, rot_dim: int, rank: int, q_rows: Optional[torch.Tensor] = None, pairs: bool = False) -> None:
     """Between the projections of a latent attention and its kernel: from fp32 rows [n, ld] (every head's ``dim`` plain and
-    ``rot_dim`` rotated query numbers at ``q_off``; the latent's ``rank`` numbers and the shared key part's ``rot_dim`` at
-    ``c_off``) the plain query parts go to ``q_plain`` [n, heads * dim], the turned ones into ``q_full``
+    ``rot_dim`` rotated query numbers at ``q_off`` (of ``q_rows`` when given); the latent's ``rank`` numbers and the shared key
+    part's ``rot_dim`` at ``c_off``; rotated numbers turn with their neighbour's when ``pairs``, else with the one rot_dims/2 on) the plain query parts go to ``q_plain`` [n, heads * dim], the turned ones into ``q_full``
     [n, heads, rank + rot_dim] behind each head's first ``rank`` places, and (normed latent, turned key part) into the
     pages [pages, 1, page_size, rank + rot_dim] at ``slots``."""
     if rows.dtype != torch.float32 or not rows.is_cuda or rows.stride(1) != 1:
         raise KernelError("latent prep: fp32 rows with unit column stride are needed")
     n = rows.shape[0]
+    q_rows = rows if q_rows is None else q_rows
+    if q_rows.dtype != torch.float32 or not q_rows.is_cuda or q_rows.stride(1) != 1 or q_rows.shape[0] != n:
+        raise KernelError("latent prep: fp32 query rows with unit column stride are needed")
     _need(q_plain, "q_plain")
     _need(q_full, "q_full", q_plain.dtype)
     _need(norm_weight, "latent norm weight")
@@ -1355,8 +1417,9 @@ def latent_prep(rows: torch.Tensor, q_off: int, c_off: int, norm_weight: torch.T
         _need(slots, "slots", torch.int32)
         if pages.shape[1:] != (1, page_size, rank + rot_dim):
             raise KernelError("latent prep: page pool shape mismatch")
-    check(_lib.load().mm_latent_prep(rows.data_ptr(), rows.stride(0), int(q_off), int(c_off), norm_weight.data_ptr(), dtype_code(norm_weight.dtype),
-                                     float(eps), _ptr(rot) if rot_dims else None, int(rot_dims), q_plain.data_ptr(), q_full.data_ptr(), _ptr(pages),
+    check(_lib.load().mm_latent_prep(q_rows.data_ptr(), q_rows.stride(0), int(q_off), rows.data_ptr(), rows.stride(0), int(c_off),
+                                     norm_weight.data_ptr(), dtype_code(norm_weight.dtype), float(eps), _ptr(rot) if rot_dims else None,
+                                     int(rot_dims), int(bool(pairs)), q_plain.data_ptr(), q_full.data_ptr(), _ptr(pages),
                                      dtype_code(q_plain.dtype), _ptr(slots) if pages is not None else None, int(page_size), n, int(heads), int(dim),
                                      int(rot_dim), int(rank), _stream()), "latent_prep")
 
@@ -1579,10 +1642,52 @@ def post_norm(residual: torch.Tensor, a: Optional[torch.Tensor], b: Optional[tor
     return out
 
 
+def output_norm(residual: torch.Tensor, a: torch.Tensor, weight: torch.Tensor, eps: float, mult: float, *, ca: float = 1.0,
+                wts: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None, cb: float = 1.0,
+                gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """``y = ca a + cb gate b``, ``x <- x + mult y / sqrt(mean(y^2) + eps) * weight`` on the fp32 residual ``x`` [n, D] in place.
+    ``a`` [n, D], or with ``wts`` (fp32 [n, top]) the rows [n * top, D] of every token's chosen experts, weighed and added here
+    (``place`` int32 [n, top] says where a row stands; None: in the order of the choice); ``b`` [n, D] or None, times ``gate``
+    fp32 [n] when given; ``out`` also gets the new rows in its own dtype."""
+    _need(residual, "residual", torch.float32)
+    _need(weight, "norm weight", torch.float32)
+    n, D = residual.shape
+    _need(a, "branch")
+    top = 0
+    if wts is not None:
+        _need(wts, "expert weights", torch.float32)
+        top = wts.shape[1]
+        if wts.shape[0] != n:
+            raise KernelError("output norm: one row of weights per token")
+        if place is not None:
+            _need(place, "places", torch.int32)
+            if place.numel() < n * top:
+                raise KernelError("output norm: one place per (token, choice)")
+    if a.shape != (n * max(1, top), D):
+        raise KernelError("output norm: a branch has another shape")
+    if b is not None:
+        _need(b, "branch")
+        if b.shape != (n, D):
+            raise KernelError("output norm: a branch has another shape")
+        if gate is not None:
+            _need(gate, "branch gate", torch.float32)
+            if gate.numel() != n:
+                raise KernelError("output norm: one gate per token")
+    if out is not None:
+        _need(out, "output norm out")
+        if out.shape != (n, D):
+            raise KernelError("output norm: out has another shape")
+    check(_lib.load().mm_output_norm(residual.data_ptr(), a.data_ptr(), dtype_code(a.dtype), _ptr(wts), _ptr(place), top, _ptr(b),
+                                     dtype_code(b.dtype) if b is not None else F32, _ptr(gate) if b is not None else None, weight.data_ptr(),
+                                     _ptr(out), dtype_code(out.dtype) if out is not None else F32, n, D, float(mult), float(ca), float(cb), float(eps),
+                                     _stream()), "output_norm")
+    return out
+
+
 def glu_rows(gate_up: torch.Tensor, out_dtype: torch.dtype, activation: str = "silu", limit: float = 0.0,
-             row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """The gated activation of rows [n, 2F] whose first F columns are the gate's and the rest the up projection's
-    (``GLU_ACTIVATIONS``), each row multiplied by ``row_scale`` [n] first when given: [n, F] of ``out_dtype``."""
+             row_scale: Optional[torch.Tensor] = None, interleave: int = 0) -> torch.Tensor:
+    """The gated activation of rows [n, 2F] whose first F columns are the gate's and the rest the up projection's, or which hold
+    both in turn in blocks of ``interleave`` columns (``GLU_ACTIVATIONS``), each row multiplied by ``row_scale`` [n] first when given: [n, F] of ``out_dtype``."""
     if not gate_up.is_cuda or gate_up.stride(1) != 1 or gate_up.shape[1] % 2:
         raise KernelError("gated activation: rows of an even width with unit column stride are needed")
     n, F2 = gate_up.shape
@@ -1590,7 +1695,7 @@ def glu_rows(gate_up: torch.Tensor, out_dtype: torch.dtype, activation: str = "s
         _need(row_scale, "row scale", torch.float32)
     out = torch.empty((n, F2 // 2), dtype=out_dtype, device=gate_up.device)
     check(_lib.load().mm_glu_rows(gate_up.data_ptr(), dtype_code(gate_up.dtype), gate_up.stride(0), out.data_ptr(), dtype_code(out_dtype), n, F2 // 2,
-                                  GLU_ACTIVATIONS[activation], float(limit), _ptr(row_scale), _stream()), "glu_rows")
+                                  GLU_ACTIVATIONS[activation], float(limit), _ptr(row_scale), int(interleave), _stream()), "glu_rows")
     return out
 
 
@@ -1602,13 +1707,18 @@ def cast_rows(x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
     return out
 
 
-def scaled_sum2(a: torch.Tensor, b: torch.Tensor, ca: float, cb: float) -> torch.Tensor:
-    """``ca * a + cb * b`` element by element."""
+def scaled_sum2(a: torch.Tensor, b: torch.Tensor, ca: float, cb: float, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``ca * a + cb * gate * b`` element by element; ``gate``: a number per row (None: 1)."""
     _need(a, "scaled sum a")
     _need(b, "scaled sum b", a.dtype)
     if a.shape != b.shape:
         raise KernelError("scaled sum: shape mismatch")
+    if gate is not None:
+        _need(gate, "scaled sum gate", torch.float32)
+        if gate.numel() != a.shape[0]:
+            raise KernelError("scaled sum: one gate per row")
     out = torch.empty_like(a)
-    check(_lib.load().mm_scaled_sum2(a.data_ptr(), b.data_ptr(), out.data_ptr(), dtype_code(a.dtype), a.numel(), float(ca), float(cb), _stream()),
+    check(_lib.load().mm_scaled_sum2(a.data_ptr(), b.data_ptr(), out.data_ptr(), dtype_code(a.dtype), a.numel(), float(ca), float(cb), _ptr(gate),
+                                     a.shape[-1], _stream()),
           "scaled_sum2")
     return out

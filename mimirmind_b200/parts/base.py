@@ -176,6 +176,19 @@ class NormedRows:
 
 
 @dataclass
+class SplitBranch:
+    """A sublayer's output still in pieces, for a block whose own launch puts them together:
+    ``sum_c weights[t, c] rows[place[t, c]] + gate[t] other[t]``.  Without ``weights`` ``rows`` is [n, width] as it stands; without
+    ``place`` a token's rows follow one another; ``other`` (and its gate) may be absent."""
+
+    rows: torch.Tensor
+    weights: Optional[torch.Tensor] = None     # fp32 [n, choices]
+    place: Optional[torch.Tensor] = None       # int32 [n * choices]
+    other: Optional[torch.Tensor] = None       # [n, width]
+    gate: Optional[torch.Tensor] = None        # fp32 [n]
+
+
+@dataclass
 class NativeDesc:
     """What the native step executor (csrc/exec) needs to build its own object of a part: the kind under which a
     C++ class is registered, numbers, tensors (as the part holds them after fusing) and the parts inside it."""

@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from ..registry import BLOCKS
-from .base import Block, FactoredRows, LayerCache, NativeDesc, NormedRows, ResidualSink, StepContext
+from .base import Block, FactoredRows, LayerCache, NativeDesc, NormedRows, ResidualSink, SplitBranch, StepContext
 
 
 @BLOCKS.register("pre_norm")
@@ -266,6 +266,59 @@ class PostNormBlock(Block):
         if ctx.dump is not None:
             dump("l_out", residual)
         return NormedRows(h) if isinstance(successor, PostNormBlock) else None
+
+
+@BLOCKS.register("output_norm")
+class OutputNormBlock(Block):
+    """A norm on each sublayer's output and none on its input: ``x <- x + m norm1(mixer(x))``, then ``x <- x + m norm2(ffn(x))``;
+    the sublayers read the stream itself, and a layer whose feed-forward is of kind ``none`` has the first sublayer only.  Both
+    norms are of the kind ``y w / sqrt(mean(y^2) + eps)`` (``Norm.factors``).
+
+    Norm, scaling and sum are one launch that leaves the fp32 stream and its rounding to the activation dtype, which is what the
+    next sublayer's products read (the block that follows, if it is of this kind, gets those rows as ``NormedRows``).  A
+    feed-forward whose result is a sum of pieces (``forward_split``) hands them over and the same launch weighs and adds them.
+
+    spec params: mult (m)."""
+
+    def __init__(self, *args, **kwargs):
+        super().__init__(*args, **kwargs)
+        from .mlp import NoFeedForward
+        self.mult = float(self.spec.get("mult", 1.0))
+        self.has_ffn = not isinstance(self.feed_forward, NoFeedForward)
+        self.norms = []
+        for norm in (self.mixer_norm,) + ((self.ffn_norm,) if self.has_ffn else ()):
+            f = norm.factors()
+            if f is None:
+                raise ValueError("output_norm block: its norms must be of the kind y * w / sqrt(mean(y^2) + eps)")
+            self.norms.append((f[0].float().contiguous(), float(f[1])))
+
+    def _add(self, residual: torch.Tensor, branch, which: int) -> torch.Tensor:
+        from ..kernels import ops
+        w, eps = self.norms[which]
+        b = branch if isinstance(branch, SplitBranch) else SplitBranch(branch)
+        out = None if self.rt.dtype == torch.float32 else torch.empty(residual.shape, dtype=self.rt.dtype, device=residual.device)
+        ops.output_norm(residual, b.rows, w, eps, self.mult, wts=b.weights, place=b.place, b=b.other, gate=b.gate, out=out)
+        return residual if out is None else out          # a float32 run reads the stream itself
+
+    def forward(self, residual: torch.Tensor, pending, ctx: StepContext, cache: LayerCache,
+                successor: Optional[Block] = None):
+        from ..kernels import ops
+        dump = ctx.dump or (lambda stage, t: None)
+        if isinstance(pending, NormedRows):
+            h = pending.x
+        else:
+            if pending is not None:
+                ops.add_residual(residual, pending)
+            h = residual if self.rt.dtype == torch.float32 else ops.cast_rows(residual, self.rt.dtype)
+        dump("attn_norm", h)
+        h = self._add(residual, self.mixer.forward(h, ctx, cache), 0)
+        dump("attn_out", residual)               # the stream behind the mixer's sublayer
+        if self.has_ffn:
+            split = getattr(self.feed_forward, "forward_split", self.feed_forward.forward)
+            h = self._add(residual, split(h, ctx), 1)
+        if ctx.dump is not None:
+            dump("l_out", residual)
+        return NormedRows(h) if isinstance(successor, OutputNormBlock) else None
 
 
 def ops_add(residual: torch.Tensor, delta: torch.Tensor) -> None:

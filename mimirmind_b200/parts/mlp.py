@@ -1,4 +1,4 @@
-"""Gated feed-forward: ``y = (act(x·Wgᵀ) ⊙ x·Wuᵀ)·Wdᵀ`` with SiLU as the activation.
+"""Gated feed-forward: ``y = (act(x·Wgᵀ) ⊙ x·Wuᵀ)·Wdᵀ`` with SiLU (or the tanh form of gelu) as the activation.
 
 No biases (src/runtime/arch/Qwen2Backend.cpp:443-458); ``silu(g) = g / (1 + exp(−g))``
 (src/compute/Activations.cpp:25-36).  Gate and up weights are concatenated at load so
@@ -19,7 +19,8 @@ from .linear import linear
 
 @FEED_FORWARDS.register("swiglu")
 class SwiGLU(FeedForward):
-    """spec params: hidden, intermediate, gate, up, down (tensor names under the prefix)."""
+    """spec params: hidden, intermediate, gate, up, down (tensor names under the prefix), activation (``silu``, the default, or
+    ``gelu_tanh``)."""
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> List[TensorSpec]:
@@ -34,6 +35,9 @@ class SwiGLU(FeedForward):
         super().__init__(spec, weights, rt)
         self.hidden = int(spec["hidden"])
         self.intermediate = int(spec["intermediate"])
+        self.activation = str(spec.get("activation", "silu"))
+        if self.activation not in ("silu", "gelu_tanh"):
+            raise ValueError("swiglu: activation is 'silu' or 'gelu_tanh'")
         gate = weights.take(spec["gate"])
         up = weights.take(spec["up"])
         if gate.dtype != up.dtype:
@@ -51,7 +55,7 @@ class SwiGLU(FeedForward):
         self.w_down = weights.take(spec["down"]).contiguous()       # [d, F]
 
     def native(self):
-        if type(self) is not SwiGLU:
+        if type(self) is not SwiGLU or self.activation != "silu":
             return None
         return NativeDesc("swiglu", {"hidden": self.hidden, "intermediate": self.intermediate, "interleave": self.interleave},
                           {"w_gate_up": self.w_gate_up, "w_down": self.w_down})
@@ -61,11 +65,16 @@ class SwiGLU(FeedForward):
             and self.w_down.dtype == torch.bfloat16 and self.rt.matmul != "simt"
 
     def fuses(self, n_tokens: int) -> bool:
+        return self.activation == "silu" and self._small(n_tokens)
+
+    def _small(self, n_tokens: int) -> bool:
         return (self._tensor_cores() and ops.small_batch_supported(n_tokens, 2 * self.intermediate, self.hidden)
                 and ops.small_batch_supported(n_tokens, self.hidden, self.intermediate))
 
     def forward(self, x, ctx: StepContext, sink: Optional[ResidualSink] = None):
         m = x.shape[0]
+        if self.activation != "silu":
+            return linear(self._hidden(x), self.w_down, None, self.rt)
         if self.fuses(m):
             # a few tokens: two weight-streaming products; 1/rms and activation in the first one's epilogue,
             # residual add and the next norm in the second one's
@@ -85,6 +94,18 @@ class SwiGLU(FeedForward):
         return linear(act, self.w_down, None, self.rt)
 
 
+    def _hidden(self, x: torch.Tensor) -> torch.Tensor:
+        """act(gate) * up for another activation than silu: in the epilogue of the weight-streaming products (a few tokens) or
+        of the tcgen05 product (prompt-sized steps), otherwise an fp32 product and a pass over it."""
+        m = x.shape[0]
+        if self._small(m):
+            return ops.gemv_bf16_glu(x, self.w_gate_up, self.activation)
+        if self._tensor_cores() and m >= ops.TCGEN05_SWIGLU_MIN_ROWS and ops.gemm_tcgen05_supported(m, 2 * self.intermediate, self.hidden):
+            return ops.gemm_tcgen05_glu(x, self.w_gate_up, self.activation)
+        gu = linear(x, self.w_gate_up, None, self.rt, out_dtype=torch.float32)
+        return ops.glu_rows(gu, self.rt.dtype, self.activation, interleave=self.interleave)
+
+
 # From this model width on the up product of a prompt portion takes its bias and activation as the epilogue of this
 # library's tcgen05 product; below it the library product and a separate pass are faster (measured, 2,048 tokens, whole
 # step of 8 layers: width 4096 / ff 16384: 4.68 against 4.71 ms; width 2048 / ff 8192: 2.46 against 2.20 ms, where the
@@ -95,7 +116,7 @@ FUSED_UP_MIN_HIDDEN = 4096
 @FEED_FORWARDS.register("dense_mlp")
 class DenseMLP(FeedForward):
     """Two-matrix feed-forward ``y = act(x·W_upᵀ + b_up)·W_downᵀ + b_down`` with the activation as a parameter
-    (``relu2``: the square of relu; ``gelu_tanh``; ``silu``; ``relu``).  Bias and activation are one fp32 pass over the
+    (``relu2``: the square of relu; ``gelu_tanh``; ``silu``; ``relu``; ``gelu_erf``, the exact form).  Bias and activation are one fp32 pass over the
     hidden rows (``csrc/bias_act.cu``).
 
     spec params: hidden, ff, activation, bias (bool), up, down (weights; biases are the name + ``bias_suffix``)."""
@@ -125,7 +146,7 @@ class DenseMLP(FeedForward):
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         if (x.dtype == torch.bfloat16 and self.w_up.dtype == torch.bfloat16 and self.rt.matmul != "simt" and not ctx.plain_only
-                and ops.gemv_supported(x.shape[0], self.ff, self.hidden)):
+                and ops.small_batch_supported(x.shape[0], self.ff, self.hidden)):
             # a few tokens: bias and activation in the epilogue of the weight-streaming product
             hidden = ops.gemv_bf16_act(x, self.w_up, self.b_up, self.activation)
             return linear(hidden, self.w_down, self.b_down, self.rt)

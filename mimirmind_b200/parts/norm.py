@@ -20,7 +20,8 @@ from .base import NativeDesc, Norm, Runtime, WeightView
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
     """spec params: width, eps, weight (tensor name under the prefix), offset (default 0: the stored weight multiplies
-    directly; 1: the weight is stored around zero and ``1 + w`` multiplies, formed once at load in fp32), streams (default
+    directly; 1: the weight is stored around zero and ``1 + w`` multiplies, formed once at load in fp32), gain (default 1: a
+    constant that multiplies the result, carried by the weight; the scale of the logits behind a final norm), streams (default
     1; S: the residual holds S streams per token, ``[n, S * width]``, and the norm is taken of their sum)."""
 
     @classmethod
@@ -33,16 +34,19 @@ class RMSNorm(Norm):
         self.eps = float(spec["eps"])
         self.offset = float(spec.get("offset", 0.0))
         self.streams = int(spec.get("streams", 1) or 1)
+        self.gain = float(spec.get("gain", 1.0))
         self.weight = weights.get(spec["weight"]).contiguous()
         if self.offset:
             self.weight = (self.weight.float() + self.offset).contiguous()
+        if self.gain != 1.0:
+            self.weight = (self.weight.float() * self.gain).contiguous()
         self._ones = torch.ones(self.streams, dtype=torch.float32, device=rt.device) if self.streams > 1 else None
 
     def factors(self):
         return (self.weight, self.eps) if self.streams == 1 else None
 
     def native(self):
-        if type(self) is not RMSNorm or self.offset or self.streams != 1:
+        if type(self) is not RMSNorm or self.offset or self.gain != 1.0 or self.streams != 1:
             return None
         return NativeDesc("rmsnorm", {"width": self.width, "eps": self.eps}, {"weight": self.weight})
 

@@ -7,11 +7,34 @@ Pairs are ``(i, i + half)``; ``angle = pos · theta^(−2i/dim)``;
 """
 from __future__ import annotations
 
-from typing import Optional, Tuple
+import math
+from typing import Any, Mapping, Optional, Tuple
+
+import torch
 
 from ..config.spec import PartSpec
 from ..registry import POSITION_ENCODINGS
 from .base import NativeDesc, PositionEncoding, Runtime, WeightView
+
+
+def exact_frequencies(base: float, dims: int, scaling: Optional[Mapping[str, Any]] = None) -> Tuple[torch.Tensor, float]:
+    """``base^(-2i/dims)`` for ``i < dims/2`` in float64, and what multiplies cos and sin.  With ``scaling`` (``factor``,
+    ``original``, ``fast``, ``slow``) YaRN's interpolation: the pair that turns ``t`` times over ``original`` positions is number
+    ``dims ln(original / (2 pi t)) / (2 ln base)``; up to the one of ``fast`` turns frequencies stay, from the one of ``slow`` turns on
+    they are divided by ``factor``, between them in proportion; cos and sin are multiplied by ``0.1 ln(factor) + 1``."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
+    if scaling is None:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def number(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    first = max(math.floor(number(float(scaling["fast"]))), 0)
+    last = min(math.ceil(number(float(scaling["slow"]))), dims - 1)
+    ramp = ((i - first) / max(last - first, 0.001)).clamp(0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
 
 
 @POSITION_ENCODINGS.register("rotary_half")
@@ -55,7 +78,6 @@ class RotaryPairs(PositionEncoding):
 
     def __init__(self, spec: PartSpec, weights: WeightView, rt: Runtime):
         super().__init__(spec, weights, rt)
-        import torch
         self.base, self.dims = float(spec["base"]), int(spec["dims"])
         if self.dims % 2 or self.dims < 0:
             raise ValueError("rotary_pairs: dims must be even")
