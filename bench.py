@@ -166,7 +166,7 @@ def run_workload(name: str, layers: int) -> int:
     return 0 if verified else 1
 
 
-# ---- another design beside the closest existing one, at equal size (--compare bigerax | domelix | tupunex | zubarax) ---------------------------------------
+# ---- another design beside the closest existing one, at equal size (--compare bigerax | domelix | segorax | tupunex | zubarax) ---------------------------------------
 # Layer sizes that resemble a real model's; both models get the same width, heads, key size, window, layer count and
 # vocabulary, and feed-forwards of equal parameter count (two matrices of ff against three of 2/3 ff).
 COMPARE_SIZES = {
@@ -234,6 +234,30 @@ def zubarax_config(z):
             "layers": layers}
 
 
+def segorax_config(z):
+    """Three layers of latent attention with low-rank queries and a sink to one with direct queries and an interpolated rotation
+    (512 + 64 numbers cached per token); the first of four feed-forwards dense, the others 16 experts of two matrices, 4 chosen from the
+    2 best of 4 groups, and a gated shared expert, with the dense one's parameters active."""
+    d, H, dk = z["width"], z["heads"], z["dim"]
+    inter, expert_ff = -(-(2 * z["ff"] // 3) // 64) * 64, -(-(z["ff"] // 5) // 64) * 64
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}}, "shared": {"ff": expert_ff}}
+    size = {"heads": H, "dim": dk, "rot_dim": 64, "vdim": dk, "kv_rank": 512, "scale": (dk + 64) ** -0.5}
+    low = dict(size, q_rank=3 * d // 8, rot={"base": 10000.0, "dims": 64})
+    far = dict(size, rot={"base": 10000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    layers = [{"type": "latent_attention_2", "mixer": far, "mlp": moe} if i % 4 == 2 else
+              {"type": "latent_attention", "mixer": low, "mlp": moe if i % 4 else {"kind": "dense", "ff": inter}} for i in range(z["layers"])]
+    return {"architecture": "Segorax", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_scale": 0.5,
+            "embedding": {"scale": 8.0}, "layers": layers}
+
+
+def tupunex_latent_config(z):
+    """Tupunex with latent attention in every layer and one residual stream: the same attention sizes and a dense feed-forward."""
+    out = tupunex_config(z)
+    out["layers"] = [out["layers"][2] if len(out["layers"]) > 2 else tupunex_config(dict(z, layers=3))["layers"][2]] * z["layers"]
+    del out["streams"]
+    return out
+
+
 def qwen2_config(z, context):
     inter = -(-(2 * z["ff"] // 3) // 64) * 64
     return dict(architectures=["Qwen2ForCausalLM"], model_type="qwen2", num_hidden_layers=z["layers"], hidden_size=z["width"],
@@ -244,7 +268,8 @@ def qwen2_config(z, context):
 
 def run_compare(args) -> int:
     """Prefill and decode throughput of one design beside the closest other one at equal size (random weights, bfloat16):
-    Bigerax beside the Qwen2 decoder, Domelix beside Bigerax, Tupunex beside the Qwen2 decoder, Zubarax beside Domelix; one prompt in one step (median of five), and the captured
+    Bigerax beside the Qwen2 decoder, Domelix beside Bigerax, Tupunex beside the Qwen2 decoder, Zubarax beside Domelix,
+    Segorax beside Tupunex with latent attention in every layer; one prompt in one step (median of five), and the captured
     decode step at the given batch over prompts of that length."""
     import numpy as np
     import torch
@@ -261,9 +286,10 @@ def run_compare(args) -> int:
     steps, warmup, batch = max(1, min(args.steps, 128)), max(3, args.warmup), max(1, args.batch)
     context = -(-(prompt_len + SETTLE_STEPS + warmup + steps + 1) // 1024) * 1024
     first, second = {"bigerax": ("bigerax", "qwen2"), "domelix": ("domelix", "bigerax"), "tupunex": ("tupunex", "qwen2"),
-                     "zubarax": ("zubarax", "domelix")}[args.compare]
+                     "zubarax": ("zubarax", "domelix"), "segorax": ("segorax", "tupunex_latent")}[args.compare]
     configs = {"bigerax": lambda z: bigerax_config(z), "qwen2": lambda z: qwen2_config(z, context), "domelix": lambda z: domelix_config(z),
-               "tupunex": lambda z: tupunex_config(z), "zubarax": lambda z: zubarax_config(z)}
+               "tupunex": lambda z: tupunex_config(z), "zubarax": lambda z: zubarax_config(z), "segorax": lambda z: segorax_config(z),
+               "tupunex_latent": lambda z: tupunex_latent_config(z)}
     out = {"compare": first, "beside": second, "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len, "batch": batch,
            "steps": steps, "warmup": warmup, "sizes": {}}
     sizes = [args.size] if args.size else sorted(COMPARE_SIZES)
@@ -383,9 +409,9 @@ def main() -> int:
                     help="with --only decode or prefill: prompts of this many tokens instead of 2,048 (the context grows with them)")
     ap.add_argument("--opt", action="append", default=[], metavar="NAME=VALUE",
                     help="set a tunable of the library's dispatch (csrc/exec/exec.h, Options) for this run, e.g. cluster_max_wanted=64")
-    ap.add_argument("--compare", default="", choices=["", "bigerax", "domelix", "tupunex", "zubarax"],
+    ap.add_argument("--compare", default="", choices=["", "bigerax", "domelix", "segorax", "tupunex", "zubarax"],
                     help="instead of the default run: prefill and decode throughput of that design beside the closest other one (bigerax "
-                         "beside the Qwen2 decoder, domelix beside bigerax, tupunex beside the Qwen2 decoder) at equal size, at layer sizes that resemble a real model's (random weights; --size, --layers, --batch, --prompt-len, --steps)")
+                         "beside the Qwen2 decoder, domelix beside bigerax, tupunex beside the Qwen2 decoder, zubarax beside domelix, segorax beside tupunex with latent attention in every layer) at equal size, at layer sizes that resemble a real model's (random weights; --size, --layers, --batch, --prompt-len, --steps)")
     ap.add_argument("--size", default="", choices=[""] + sorted(COMPARE_SIZES), help="with --compare: one size only")
     args = ap.parse_args()
 
