@@ -90,8 +90,9 @@ MM_EXPORT int mm_qkv_split_post(const void* rows, int ld, int q_off, int k_off, 
 // q_rows [n, ldq] fp32: H heads of (dk plain, dr rotated) query numbers at q_off; c_rows [n, ldc] fp32 (may be the same
 // rows): the latent's `rank` numbers and the shared key part's dr numbers at c_off.  rot [n, rot_dims / 2] (cos, sin);
 // number i turns with i + rot_dims / 2, or with `pairs` 2i with 2i + 1; numbers from rot_dims on of a rotated part pass.
-// q_plain [n, H, dk]; q_full [n, H, rank + dr] gets each head's rotated part at [rank, rank + dr); pages
-// [pages, 1, page_size, rank + dr] get (normed latent, rotated key part).
+// q_plain [n, H, dk]; q_full [n, H, rank + dr] gets each head's rotated part at [rank, rank + dr) (both null: not wanted); pages
+// [pages, 1, page_size, rank + dr] get (normed latent, rotated key part).  q_wide [n, H, wide_w] or null: each head's plain part
+// at 0, zeros from dk on, the rotated part at wide_rot, zeros behind it (dk, dr, wide_rot and wide_w multiples of 8).
 __device__ __forceinline__ float turned(const float* part, const float2* rt, int e, int rot_dims, int pairs) {
     if (e >= rot_dims) return part[e];
     const int half = rot_dims >> 1;
@@ -105,7 +106,7 @@ template <typename T>
 __global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, int q_off, const float* __restrict__ c_rows, int ldc, int c_off,
                                    const void* __restrict__ norm_w, int w_dtype, float eps, const float2* __restrict__ rot, int rot_dims, int pairs,
                                    T* __restrict__ q_plain, T* __restrict__ q_full, T* __restrict__ pages, const int32_t* __restrict__ slots,
-                                   int page_size, int H, int dk, int dr, int rank) {
+                                   int page_size, int H, int dk, int dr, int rank, T* __restrict__ q_wide, int wide_rot, int wide_w) {
     __shared__ float scratch[32];
     const int t = blockIdx.x;
     const float* row = q_rows + (size_t)t * ldq;
@@ -114,11 +115,29 @@ __global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, in
     const float2* rt = rot + (size_t)t * half;
     const int wide = rank + dr;
     // queries: plain parts to their buffer, rotated parts into the joined query
-    for (int i = threadIdx.x; i < H * dk; i += blockDim.x) {
+    if (q_wide != nullptr) {
+        const int per = wide_w / 8;
+        for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+            const int h = i / per, e0 = (i - h * per) * 8;
+            const float* head = row + q_off + h * (dk + dr);
+            __align__(16) T v[8];
+            if (e0 < wide_rot) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] = from_f32<T>(e0 < dk ? head[e0 + j] : 0.0f);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] = from_f32<T>(e0 - wide_rot < dr ? turned(head + dk, rt, e0 - wide_rot + j, rot_dims, pairs) : 0.0f);
+            }
+            T* dst = q_wide + ((size_t)t * H + h) * wide_w + e0;
+#pragma unroll
+            for (int j = 0; j < (int)sizeof(v) / 16; ++j) reinterpret_cast<uint4*>(dst)[j] = reinterpret_cast<const uint4*>(v)[j];
+        }
+    }
+    for (int i = threadIdx.x; q_plain != nullptr && i < H * dk; i += blockDim.x) {
         const int h = i / dk, e = i - h * dk;
         q_plain[(size_t)t * H * dk + i] = from_f32<T>(row[q_off + h * (dk + dr) + e]);
     }
-    for (int i = threadIdx.x; i < H * dr; i += blockDim.x) {
+    for (int i = threadIdx.x; q_full != nullptr && i < H * dr; i += blockDim.x) {
         const int h = i / dr, e = i - h * dr;
         q_full[((size_t)t * H + h) * wide + rank + e] = from_f32<T>(turned(row + q_off + h * (dk + dr) + dk, rt, e, rot_dims, pairs));
     }
@@ -139,20 +158,24 @@ __global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, in
 
 MM_EXPORT int mm_latent_prep(const void* q_rows, int ldq, int q_off, const void* c_rows, int ldc, int c_off, const void* norm_w, int w_dtype,
                              float eps, const void* rot, int rot_dims, int pairs, void* q_plain, void* q_full, void* pages, int dtype, const void* slots, int page_size, int n_tokens,
-                             int H, int dk, int dr, int rank, void* stream) {
+                             int H, int dk, int dr, int rank, void* q_wide, int wide_rot, int wide_w, void* stream) {
     MM_REQUIRE(n_tokens >= 0 && H > 0 && dk > 0 && dr >= 0 && rank > 0, "latent prep: bad sizes");
     MM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dr && (rot_dims == 0 || rot != nullptr), "latent prep: the rotated dimensions are even and at most the rotated part");
     MM_REQUIRE(q_off >= 0 && c_off >= 0 && ldq >= q_off + H * (dk + dr) && ldc >= c_off + rank + dr, "latent prep: the rows are narrower than what is cut out of them");
     MM_REQUIRE(pages == nullptr || (slots != nullptr && page_size > 0), "latent prep: bad page geometry");
+    MM_REQUIRE((q_plain == nullptr) == (q_full == nullptr) && (q_plain != nullptr || q_wide != nullptr), "latent prep: nowhere to put the queries");
+    MM_REQUIRE(q_wide == nullptr || (dk % 8 == 0 && dr % 8 == 0 && wide_rot % 8 == 0 && wide_w % 8 == 0 && dk <= wide_rot && wide_rot + dr <= wide_w &&
+                                     ((uintptr_t)q_wide & 15) == 0), "latent prep: wide queries need parts of multiples of 8 that fit their places");
     if (n_tokens == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == MM_F32)
         mm_launch(latent_prep_kernel<float>, dim3(n_tokens), dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
-                  norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (float*)q_plain, (float*)q_full, (float*)pages, (const int32_t*)slots, page_size, H, dk, dr, rank);
+                  norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (float*)q_plain, (float*)q_full, (float*)pages, (const int32_t*)slots, page_size, H, dk, dr, rank,
+                  (float*)q_wide, wide_rot, wide_w);
     else if (dtype == MM_BF16)
         mm_launch(latent_prep_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
                   norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_full, (__nv_bfloat16*)pages, (const int32_t*)slots,
-                  page_size, H, dk, dr, rank);
+                  page_size, H, dk, dr, rank, (__nv_bfloat16*)q_wide, wide_rot, wide_w);
     else
         MM_REQUIRE(false, "latent prep: dtype must be float32 or bfloat16");
     MM_CHECK_LAUNCH();

@@ -27,7 +27,7 @@
 // ring), which nothing of that needs.
 // All mbarrier waits are bounded; on a time-out the kernel frees its tensor memory, sets `err`
 // and returns.
-#include "tcgen05.cuh"
+#include "tcgen05_attention.cuh"
 
 namespace {
 
@@ -45,7 +45,6 @@ constexpr int SOFTMAX_WARPS = 8;               // two groups of four
 constexpr int GROUP_WARPS = 4;                 // barriers between the softmax warps and the tensor core count warps, not
                                                // threads: one arrival per softmax warp on one mbarrier serialise and cost more than the math
 constexpr int TMEM_COLS_ATT = 512;              // S of the even / odd tiles: columns 0..255; O of the even / odd tiles: from 256, head-size columns each
-constexpr float RESCALE_STEP = 8.0f;            // log2 of how far a row's maximum may run ahead of its reference
 
 struct AttCtl {
     uint64_t q_full;
@@ -63,49 +62,6 @@ struct AttCtl {
     uint64_t l_full;         // both groups have posted each row's reference maximum and sum (one arrival per softmax warp)
     float xchg[2][2][128];   // [group][maximum, sum][row]
 };
-
-__device__ __forceinline__ void tmem_ld32_nowait(uint32_t taddr, uint32_t* r) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
-        "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-          "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-          "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-          "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-        : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t* r) {
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-                   "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-                 : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
-                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]),
-                   "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-                 : "memory");
-}
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-
-// 2^x on the special-function unit in one instruction (relative error 2^-22, far below the bf16 rounding of P)
-__device__ __forceinline__ float fast_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
-__device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
-    __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<uint32_t*>(&v);
-}
-
-// Every lane has done its part (and its fences); one lane arrives for the warp.
-__device__ __forceinline__ void warp_arrive(uint32_t bar, int lane) {
-    __syncwarp();
-    if (lane == 0) mbar_arrive(bar);
-}
 
 // tiles: int32 [n_tiles, 4] = (request index, first token row, rows in the tile (<= 128), position of the first row)
 template <int HD>
@@ -294,78 +250,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
         uint32_t done = 0;                 // tiles of this group so far
         bool ok = true;
         uint32_t sreg[128];
+        const SoftmaxBars bars = {smem_u32(&ctl->s_full[g]), smem_u32(&ctl->s_free[g]), smem_u32(&ctl->p_full[g]), smem_u32(&ctl->pv_done[g])};
         for (uint32_t it = g; (int)it < n_tiles_k && ok; it += 2, ++done) {
-            const int kt = kt_begin + (int)it;
-            const uint32_t u = it >> 1;
-            if (!mbar_wait(smem_u32(&ctl->s_full[g]), u & 1, abort_flag)) { ok = false; break; }
-            tc_fence_after();
-#pragma unroll
-            for (int c = 0; c < 4; ++c) tmem_ld32_nowait(s_addr + c * 32, sreg + c * 32);
-            tmem_ld_wait();
-            tc_fence_before();
-            warp_arrive(smem_u32(&ctl->s_free[g]), lane);  // S of this tile is in registers
-            const int key0 = kt * BN;
-            // a tile every key of which this row sees needs no mask
-            const bool interior = row_valid && key0 + BN - 1 <= pos && key0 >= wlo;
-            float mx = -INFINITY;
-            if (interior) {
-#pragma unroll
-                for (int i = 0; i < BN; ++i) mx = fmaxf(mx, __uint_as_float(sreg[i]));
-            } else {
-#pragma unroll
-                for (int i = 0; i < BN; ++i) {
-                    const int key = key0 + i;
-                    if (!(row_valid && key <= pos && key >= wlo)) sreg[i] = 0xff800000u;      // -inf
-                    mx = fmaxf(mx, __uint_as_float(sreg[i]));
-                }
-            }
-            // P V of the group's previous tile is done: its P buffer is free and its O is at rest until this tile's P
-            // is published
-            if (done >= 1 && !mbar_wait(smem_u32(&ctl->pv_done[g]), (u - 1) & 1, abort_flag)) { ok = false; break; }
-            // Move the reference only when the maximum has outgrown it by RESCALE_STEP (or there was none).  O of a
-            // row without a reference is still zero.
-            const bool move = mx > m_ref && (m_ref == -INFINITY || (mx - m_ref) * scale_log2 > RESCALE_STEP);
-            const bool scale_o = move && m_ref != -INFINITY;
-            if (__any_sync(0xffffffffu, scale_o)) {
-                tc_fence_after();
-                const float alpha = scale_o ? fast_exp2((m_ref - mx) * scale_log2) : 1.0f;
-#pragma unroll 1
-                for (int c = 0; c < HD / 16; ++c) {
-                    uint32_t oreg[16];
-                    tmem_ld16(o_addr + c * 16, oreg);
-                    tmem_ld_wait();
-#pragma unroll
-                    for (int i = 0; i < 16; ++i) oreg[i] = __float_as_uint(__uint_as_float(oreg[i]) * alpha);
-                    tmem_st16(o_addr + c * 16, oreg);
-                }
-                tmem_st_wait();
-                l *= alpha;
-            }
-            if (move) m_ref = mx;
-            const float use = (m_ref == -INFINITY) ? 0.0f : m_ref * scale_log2;
-            // probabilities, rounded to bf16 as the tensor core will read them: the row of P is two halves of 64 keys,
-            // each 8 chunks of 16 bytes, chunk index xor-ed with row % 8
-            float sum = 0.0f;
-#pragma unroll
-            for (int hf = 0; hf < 2; ++hf) {
-                unsigned char* prow = sP + g * TILE_BYTES + hf * HALF_BYTES + row * 128;
-#pragma unroll
-                for (int ch = 0; ch < 8; ++ch) {
-                    uint32_t packed[4];
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const float p0 = fast_exp2(fmaf(__uint_as_float(sreg[hf * 64 + ch * 8 + 2 * i]), scale_log2, -use));
-                        const float p1 = fast_exp2(fmaf(__uint_as_float(sreg[hf * 64 + ch * 8 + 2 * i + 1]), scale_log2, -use));
-                        sum += p0 + p1;
-                        packed[i] = pack_bf16x2(p0, p1);
-                    }
-                    *reinterpret_cast<uint4*>(prow + ((ch ^ (row & 7)) << 4)) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
-                }
-            }
-            l += sum;
-            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");      // P is read by the tensor core (async proxy)
-            tc_fence_before();                                                // ... and O, if it was rescaled, is in tensor memory
-            warp_arrive(smem_u32(&ctl->p_full[g]), lane);
+            ok = softmax_tile<HD>(bars, abort_flag, s_addr, o_addr, sP + g * TILE_BYTES, HALF_BYTES, row, lane, row_valid, pos, wlo,
+                                  (kt_begin + (int)it) * BN, it >> 1, done == 0, scale_log2, sreg, m_ref, l);
         }
         // Merge the two groups: every thread posts its row's (reference, sum); the row's output is
         // (O0 f0 + O1 f1) / (l0 f0 + l1 f1) with f = 2^((m_g - m) scale); group g writes its half of the output columns.

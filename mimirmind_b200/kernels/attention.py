@@ -8,6 +8,9 @@ src/compute/cuda/GpuOps.cpp:2711-2731).
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
+from typing import Optional, Tuple
+
 import torch
 
 from . import ops
@@ -196,16 +199,19 @@ def _latent_lib():
     return _lib.load()
 
 
-def latent_plan(ctx, num_heads: int, tile_rows: int = LATENT_TILE_ROWS):
+def latent_plan(ctx, num_heads: int, tile_rows: int = LATENT_TILE_ROWS, without=()):
     """The step's (token, head) pairs cut once, on the host, into tiles of at most ``tile_rows`` rows of one request:
     several tokens with all their heads, or one token with a slice of its heads.  A tile names tokens, not positions
-    (the kernel reads those from the device), so a captured step replays the same plan.  Returns (tiles [n, 5], n)."""
-    key = ("latent_attention_plan", num_heads, tile_rows)
+    (the kernel reads those from the device), so a captured step replays the same plan.  ``without``: requests that another
+    kernel takes.  Returns (tiles [n, 5], n)."""
+    key = ("latent_attention_plan", num_heads, tile_rows, without)
     plan = ctx.plans.get(key)
     if plan is None:
         tiles = []
         per = max(1, tile_rows // num_heads)
         for r in range(ctx.n_requests):
+            if r in without:
+                continue
             s, n, kv = ctx.q_start[r], ctx.q_len[r], ctx.kv_len[r]
             for off in range(0, n, per):
                 tokens = min(per, n - off)
@@ -218,18 +224,107 @@ def latent_plan(ctx, num_heads: int, tile_rows: int = LATENT_TILE_ROWS):
     return plan
 
 
-def paged_latent_attention(q, pages, cache, out, ctx, num_heads: int, wide: int, rank: int, window: int, scale: float, sink=None) -> torch.Tensor:
+USE_LATENT_EXPANDED = True         # False: portions of prompts run the absorbed form too (tests run both)
+LATENT_EXPANDED_MIN = 64           # tokens of a portion from which its keys and values are made in full: per cached row the
+                                   # up-projections cost what two dozen tokens' absorbed products cost more than the plain ones
+LATENT_EXPANDED_MAX_BYTES = 1 << 29    # of keys and values a step may make
+_expanded_declared = False
+
+
+def _expanded_lib():
+    global _expanded_declared
+    from ctypes import c_float, c_int, c_void_p
+    from . import lib as _lib
+    if not _expanded_declared:
+        P, I, F = c_void_p, c_int, c_float
+        _lib.declare("mm_attention_latent_tcgen05_supported", [I, I, I])
+        _lib.declare("mm_attention_latent_tcgen05_query_width", [I, I])
+        _lib.declare("mm_attention_latent_tcgen05", [P, P, P, P, P, I, I, I, I, I, I, I, F, P, P, P])
+        _lib.declare("mm_latent_gather", [P, P, I, I, P, I, I, I, I, P, P, P])
+        _expanded_declared = True
+    return _lib.load()
+
+
+def latent_expanded_supported(key_dim: int, rot_dim: int, value_dim: int, rank: int, scale: float) -> bool:
+    return rank % 8 == 0 and scale > 0 and bool(_expanded_lib().mm_attention_latent_tcgen05_supported(key_dim, rot_dim, value_dim))
+
+
+def latent_query_width(key_dim: int, rot_dim: int) -> int:
+    return int(_expanded_lib().mm_attention_latent_tcgen05_query_width(key_dim, rot_dim))
+
+
+@dataclass
+class LatentExpandedPlan:
+    """The requests of a step whose keys and values are made in full."""
+
+    requests: Tuple[int, ...]
+    rows: int                      # their cached tokens together
+    meta: torch.Tensor             # int32 [requests, 3] = (request, its first row, its rows)
+    tiles: torch.Tensor            # int32 [n, 4]
+    n_tiles: int
+    everything: bool               # no other request in the step
+    staged: Tuple[torch.Tensor, ...] = ()
+
+
+def latent_expanded_plan(ctx, row_bytes: int) -> Optional[LatentExpandedPlan]:
+    """Portions of at least LATENT_EXPANDED_MIN tokens, as long as the step's keys and values (``row_bytes`` per cached token) stay
+    within bounds; None when the step has none.  Cut once per step and shared by its layers."""
+    if not USE_LATENT_EXPANDED or ctx.max_q_len < LATENT_EXPANDED_MIN:
+        return None
+    key = ("latent_expanded_plan", row_bytes)
+    if key not in ctx.plans:
+        meta, tiles, rows = [], [], 0
+        for r in range(ctx.n_requests):
+            s, n, kv = ctx.q_start[r], ctx.q_len[r], ctx.kv_len[r]
+            if n < LATENT_EXPANDED_MIN or (rows + kv) * row_bytes > LATENT_EXPANDED_MAX_BYTES:
+                continue
+            meta.append((r, rows, kv))
+            for off in range(0, n, 128):
+                tiles.append((s + off, min(128, n - off), kv - n + off, rows))
+            rows += kv
+        plan = None
+        if meta:
+            tiles.sort(key=lambda t: t[1] + t[2])          # the kernel starts the last (longest) tiles first
+            staged = (torch.tensor(meta, dtype=torch.int32).pin_memory(), torch.tensor(tiles, dtype=torch.int32).pin_memory())
+            on_device = [t.to(ctx.positions.device, non_blocking=True) for t in staged]
+            plan = LatentExpandedPlan(tuple(m[0] for m in meta), rows, on_device[0], on_device[1], len(tiles), len(meta) == ctx.n_requests, staged)
+        ctx.plans[key] = plan
+    return ctx.plans[key]
+
+
+def latent_expanded_attention(plan: LatentExpandedPlan, q_wide, pages, cache, w_kv, out, num_heads: int, key_dim: int, rot_dim: int, value_dim: int,
+                              rank: int, scale: float, sink, rt) -> torch.Tensor:
+    """The plan's requests: their cached latents side by side, every head's plain keys and values from them in one product
+    (``w_kv`` [heads * (key_dim + value_dim), rank]), and the attention; writes those requests' rows of ``out`` [n, heads * value_dim]."""
+    from ..parts.linear import linear
+    from .lib import check
+    lib, dev = _expanded_lib(), q_wide.device
+    c = torch.empty((plan.rows, rank), dtype=torch.bfloat16, device=dev)
+    turned = torch.empty((plan.rows, rot_dim), dtype=torch.bfloat16, device=dev) if rot_dim else None
+    check(lib.mm_latent_gather(pages.data_ptr(), cache.block_table.data_ptr(), cache.block_table.shape[1], cache.page_size, plan.meta.data_ptr(),
+                               len(plan.requests), plan.rows, rank + rot_dim, rank, c.data_ptr(), turned.data_ptr() if rot_dim else None,
+                               ops._stream()), "latent_gather")
+    kv = linear(c, w_kv, None, rt)
+    check(lib.mm_attention_latent_tcgen05(q_wide.data_ptr(), kv.data_ptr(), turned.data_ptr() if rot_dim else None, out.data_ptr(), plan.tiles.data_ptr(),
+                                          plan.n_tiles, q_wide.shape[0], plan.rows, num_heads, key_dim, rot_dim, value_dim, float(scale),
+                                          sink.data_ptr() if sink is not None else None, ops.tcgen05_error_flag(dev).data_ptr(), ops._stream()),
+          "attention_latent_tcgen05")
+    return out
+
+
+def paged_latent_attention(q, pages, cache, out, ctx, num_heads: int, wide: int, rank: int, window: int, scale: float, sink=None,
+                           without=()) -> torch.Tensor:
     """Attention of ``num_heads`` query heads of ``wide`` numbers over one shared key head ``pages`` [pages, 1, page, wide]
     whose leading ``rank`` numbers are the value, with a learned ``sink`` per head (fp32 [num_heads], or None) in the softmax's
     denominator; ``out`` [n, num_heads * rank].  bfloat16 with a rank the tensor-core
     kernel is built for: that kernel, its key tiles shared out over several CTAs while the step has few query tiles;
-    anything else: the fp32-arithmetic kernel."""
+    anything else: the fp32-arithmetic kernel.  ``without``: requests whose rows somebody else makes (they may be left unwritten)."""
     if USE_LATENT_MMA and q.dtype == torch.bfloat16 and scale > 0 and _latent_lib().mm_attention_latent_supported(wide, rank):
         from .lib import check
         lib = _latent_lib()
         # portions of prompts: tiles of 64 rows (two 16-row tiles per warp, half the key traffic per row) where they fit
         tile_rows = 64 if USE_LATENT_WIDE_TILES and ctx.max_q_len * num_heads >= 64 and lib.mm_attention_latent_tile_rows(wide) == 64 else LATENT_TILE_ROWS
-        tiles, n_tiles = latent_plan(ctx, num_heads, tile_rows)
+        tiles, n_tiles = latent_plan(ctx, num_heads, tile_rows, without)
         keys = min(window, ctx.max_kv_len) if window > 0 else ctx.max_kv_len
         splits = 1
         if n_tiles < SINK_TARGET_CTAS // 2:

@@ -81,7 +81,7 @@ _PROTOTYPES = {
     "mm_hc_write": [P, P, I, P, P, P, P, P, I, F, P, I, I, I, I, P],
     "mm_rope_half_table": [P, P, P, P, I, I, F, P],
     "mm_qkv_split_post": [P, I, I, I, I, P, P, P, I, P, I, I, I, I, I, I, I, P],
-    "mm_latent_prep": [P, I, I, P, I, I, P, I, F, P, I, I, P, P, P, I, P, I, I, I, I, I, I, P],
+    "mm_latent_prep": [P, I, I, P, I, I, P, I, F, P, I, I, P, P, P, I, P, I, I, I, I, I, I, P, I, I, P],
     "mm_head_matmul": [P, c_longlong, I, P, P, c_longlong, I, I, I, I, I, I, P],
     "mm_head_finish": [P, I, I, F, I, F, F, P, I, P, I, I, I, I, I, P],
     "mm_moe_router_scored": [P, I, I, P, I, I, I, I, I, I, I, P, P, P],

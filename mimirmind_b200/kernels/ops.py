@@ -1390,38 +1390,49 @@ def qkv_split_post(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out
 
 
 def latent_prep(rows: torch.Tensor, q_off: int, c_off: int, norm_weight: torch.Tensor, eps: float, rot: Optional[torch.Tensor], rot_dims: int,
-                q_plain: torch.Tensor, q_full: torch.Tensor, pages: Optional[torch.Tensor], slots: Optional[torch.Tensor], page_size: int,
-                heads: int, dim: int, rot_dim: int, rank: int, q_rows: Optional[torch.Tensor] = None, pairs: bool = False) -> None:
+                q_plain: Optional[torch.Tensor], q_full: Optional[torch.Tensor], pages: Optional[torch.Tensor], slots: Optional[torch.Tensor],
+                page_size: int, heads: int, dim: int, rot_dim: int, rank: int, q_rows: Optional[torch.Tensor] = None, pairs: bool = False,
+                q_wide: Optional[torch.Tensor] = None, wide_rot: int = 0) -> None:
     """Between the projections of a latent attention and its kernel: from fp32 rows [n, ld] (every head's ``dim`` plain and
     ``rot_dim`` rotated query numbers at ``q_off`` (of ``q_rows`` when given); the latent's ``rank`` numbers and the shared key
     part's ``rot_dim`` at ``c_off``; rotated numbers turn with their neighbour's when ``pairs``, else with the one rot_dims/2 on) the plain query parts go to ``q_plain`` [n, heads * dim], the turned ones into ``q_full``
-    [n, heads, rank + rot_dim] behind each head's first ``rank`` places, and (normed latent, turned key part) into the
-    pages [pages, 1, page_size, rank + rot_dim] at ``slots``."""
+    [n, heads, rank + rot_dim] behind each head's first ``rank`` places (both None: not wanted), and (normed latent, turned key part)
+    into the pages [pages, 1, page_size, rank + rot_dim] at ``slots``.  ``q_wide`` [n, heads * W] gets every head's plain part at 0 and its
+    turned part at ``wide_rot``, zeros between and behind."""
     if rows.dtype != torch.float32 or not rows.is_cuda or rows.stride(1) != 1:
         raise KernelError("latent prep: fp32 rows with unit column stride are needed")
     n = rows.shape[0]
     q_rows = rows if q_rows is None else q_rows
     if q_rows.dtype != torch.float32 or not q_rows.is_cuda or q_rows.stride(1) != 1 or q_rows.shape[0] != n:
         raise KernelError("latent prep: fp32 query rows with unit column stride are needed")
-    _need(q_plain, "q_plain")
-    _need(q_full, "q_full", q_plain.dtype)
+    dt = (q_plain if q_plain is not None else q_wide).dtype
     _need(norm_weight, "latent norm weight")
-    if q_plain.shape != (n, heads * dim) or q_full.shape != (n, heads * (rank + rot_dim)) or norm_weight.numel() != rank:
+    if q_plain is not None:
+        _need(q_plain, "q_plain", dt)
+        _need(q_full, "q_full", dt)
+        if q_plain.shape != (n, heads * dim) or q_full.shape != (n, heads * (rank + rot_dim)):
+            raise KernelError("latent prep: shape mismatch")
+    if q_wide is not None:
+        _need(q_wide, "q_wide", dt)
+        if q_wide.shape[0] != n or q_wide.shape[1] % heads:
+            raise KernelError("latent prep: shape mismatch")
+    if norm_weight.numel() != rank:
         raise KernelError("latent prep: shape mismatch")
     if rot_dims:
         _need(rot, "rotation table", torch.float32)
         if rot.shape != (n, rot_dims // 2, 2):
             raise KernelError("latent prep: rotation table of another shape")
     if pages is not None:
-        _need(pages, "latent pages", q_plain.dtype)
+        _need(pages, "latent pages", dt)
         _need(slots, "slots", torch.int32)
         if pages.shape[1:] != (1, page_size, rank + rot_dim):
             raise KernelError("latent prep: page pool shape mismatch")
     check(_lib.load().mm_latent_prep(q_rows.data_ptr(), q_rows.stride(0), int(q_off), rows.data_ptr(), rows.stride(0), int(c_off),
                                      norm_weight.data_ptr(), dtype_code(norm_weight.dtype), float(eps), _ptr(rot) if rot_dims else None,
-                                     int(rot_dims), int(bool(pairs)), q_plain.data_ptr(), q_full.data_ptr(), _ptr(pages),
-                                     dtype_code(q_plain.dtype), _ptr(slots) if pages is not None else None, int(page_size), n, int(heads), int(dim),
-                                     int(rot_dim), int(rank), _stream()), "latent_prep")
+                                     int(rot_dims), int(bool(pairs)), _ptr(q_plain), _ptr(q_full), _ptr(pages),
+                                     dtype_code(dt), _ptr(slots) if pages is not None else None, int(page_size), n, int(heads), int(dim),
+                                     int(rot_dim), int(rank), _ptr(q_wide), int(wide_rot), q_wide.shape[1] // heads if q_wide is not None else 0,
+                                     _stream()), "latent_prep")
 
 
 HEAD_MATMUL_LIBRARY_FROM = 64      # rows from which the per-head products of bfloat16 rows are one batched library product

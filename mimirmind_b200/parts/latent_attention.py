@@ -15,6 +15,10 @@ Only ``c`` and the rotated key part are cached, as one per-token array of ``rank
 absorbed: ``q_plain . Wuk_h c = (Wuk_h^T q_plain) . c``, so the kernel runs H query heads of size ``rank + dr`` over ONE
 key head, whose first ``rank`` numbers are also the value; the per-head ``Wuv_h`` is applied to the attention's
 ``rank``-wide result afterwards.  Both absorbed products are a matrix per head (``head_matmul``).
+
+Portions of prompts in bfloat16 take the other way where the sizes allow it: the plain keys and the values of the request's cached
+tokens are made in full, one product over the cached latents, and the attention runs over them on tensor memory
+(``csrc/attention_latent_tcgen05.cu``): ``dk + dr + dv`` multiplications per pair and head instead of ``2 rank + dr``.
 """
 from __future__ import annotations
 
@@ -97,6 +101,12 @@ class LatentAttention(Mixer):
         # a matrix per head, [K, N] each: the key up-projection as it stands (dk -> rank), the value's transposed (rank -> dv)
         self.m_key = up_k.reshape(H, dk, r).to(act or up_k.dtype).contiguous()
         self.m_value = up_v.reshape(H, dv, r).transpose(1, 2).to(act or up_v.dtype).contiguous()
+        self.w_kv, self.q_wide = None, 0
+        if rt.dtype == torch.bfloat16 and rt.matmul != "simt" and up_k.dtype == up_v.dtype == torch.bfloat16:
+            from ..kernels import attention as attn_kernels
+            if attn_kernels.latent_expanded_supported(dk, dr, dv, r, self.scale):
+                self.w_kv = torch.cat([up_k, up_v], dim=0).contiguous()      # [H dk, then H dv, rank]
+                self.q_wide = attn_kernels.latent_query_width(dk, dr)
         self.w_o = weights.take(spec["o"]).contiguous()
 
     def kv_cache_spec(self) -> Optional[KVCacheSpec]:
@@ -123,16 +133,26 @@ class LatentAttention(Mixer):
         if self.q_rank:
             latent_q = ops.gated_group_norm(a[:, :self.q_rank], 1, self.q_rank, self.rt.dtype, eps=self.eps, weight=self.q_norm)
             q_rows = linear(latent_q, self.w_q_up, None, self.rt, out_dtype=torch.float32)
-        q_plain = torch.empty((n, H * dk), dtype=self.rt.dtype, device=a.device)
-        q_full = torch.empty((n, H * wide), dtype=self.rt.dtype, device=a.device)
-        ops.latent_prep(a, 0, self.c_off, self.norm_weight, self.eps, rot, self.rot_dims, q_plain, q_full, pages if cache.writes else None,
-                        slots, cache.page_size, H, dk, dr, r, q_rows=q_rows, pairs=self.rot_pairs)
-        ops.head_matmul(q_plain, self.m_key, q_full, H)                      # each head's first `rank` places: Wuk_h^T q_plain
-        att = torch.empty((n, H * r), dtype=self.rt.dtype, device=a.device)
         from ..kernels import attention as attn_kernels
-        attn_kernels.paged_latent_attention(q_full, pages, cache, att, ctx, H, wide, r, 0, self.scale, sink=self.sink)
+        expanded = attn_kernels.latent_expanded_plan(ctx, 2 * H * (dk + dv)) if self.w_kv is not None else None
+        absorbed = expanded is None or not expanded.everything
+        q_plain = q_full = q_wide = None
+        if absorbed:
+            q_plain = torch.empty((n, H * dk), dtype=self.rt.dtype, device=a.device)
+            q_full = torch.empty((n, H * wide), dtype=self.rt.dtype, device=a.device)
+        if expanded is not None:
+            q_wide = torch.empty((n, H * self.q_wide), dtype=self.rt.dtype, device=a.device)
+        ops.latent_prep(a, 0, self.c_off, self.norm_weight, self.eps, rot, self.rot_dims, q_plain, q_full, pages if cache.writes else None,
+                        slots, cache.page_size, H, dk, dr, r, q_rows=q_rows, pairs=self.rot_pairs, q_wide=q_wide, wide_rot=-(-dk // 64) * 64)
         o = torch.empty((n, H * dv), dtype=self.rt.dtype, device=a.device)
-        ops.head_matmul(att, self.m_value, o, H)
+        if absorbed:
+            ops.head_matmul(q_plain, self.m_key, q_full, H)                      # each head's first `rank` places: Wuk_h^T q_plain
+            att = torch.empty((n, H * r), dtype=self.rt.dtype, device=a.device)
+            attn_kernels.paged_latent_attention(q_full, pages, cache, att, ctx, H, wide, r, 0, self.scale, sink=self.sink,
+                                                without=expanded.requests if expanded is not None else ())
+            ops.head_matmul(att, self.m_value, o, H)
+        if expanded is not None:                                                 # these requests' rows of `o`
+            attn_kernels.latent_expanded_attention(expanded, q_wide, pages, cache, self.w_kv, o, H, dk, dr, dv, r, self.scale, self.sink, self.rt)
         if self.has_gate:
             o = ops.head_finish(o, H, dv, gate=a[:, self.g_off:self.g_off + H])
         return linear(o, self.w_o, None, self.rt)

@@ -94,12 +94,16 @@ def plain_mixer(x, w, layer, eps):
     return ps.latent_attention(x, w, "mix.", layer["mixer"], eps, list(range(len(x))), low, low)
 
 
-@pytest.fixture(params=["tensor-cores", "fp32-arithmetic"])
+@pytest.fixture(params=["tensor-memory", "absorbed", "fp32-arithmetic"])
 def route(request, monkeypatch):
-    """Sizes the tensor-core kernels take run them, or never."""
+    """Long portions over keys and values made in full (sizes that kernel takes), always the absorbed form on the tensor cores, or
+    the fp32-arithmetic kernel only."""
     from mimirmind_b200.kernels import attention
-    monkeypatch.setattr(attention, "USE_LATENT_MMA", request.param == "tensor-cores")
-    return request.param
+    monkeypatch.setattr(attention, "USE_LATENT_EXPANDED", request.param == "tensor-memory")
+    monkeypatch.setattr(attention, "USE_LATENT_MMA", request.param != "fp32-arithmetic")
+    yield request.param
+    from mimirmind_b200.kernels import ops
+    ops.check_tcgen05_errors(torch.device(DEV))
 
 
 MIXERS_ALONE = {
@@ -112,6 +116,8 @@ MIXERS_ALONE = {
     "far, sizes of tiles": su.far(3, 128, 64, 64, 192, 0.07, 10000.0, (8.0, 96, 32.0, 1.0), None),
     "far, narrow": su.far(5, 16, 16, 8, 64, 0.3, 300.0, (4.0, 100, 8.0, 1.0), None),
     "far, wide": su.far(2, 160, 32, 136, 64, 0.07, 7000.0, (3.0, 300, 20.0, 2.0), None),
+    "far, four pieces": su.far(3, 136, 64, 120, 96, 0.07, 7000.0, (3.0, 300, 20.0, 2.0), None),
+    "far, two rotated pieces": su.far(5, 8, 72, 56, 40, 0.12, 900.0, (6.0, 150, 30.0, 1.0), None),
 }
 
 
@@ -120,7 +126,7 @@ MIXERS_ALONE = {
 def test_latent_attention_alone(name, dtype, route):
     """One mixer, three requests: a long prompt whole, then portions of several sizes beside single tokens of others, over pages
     of their own in a pool full of NaN."""
-    if dtype == "float32" and route != "tensor-cores":
+    if dtype == "float32" and route != "tensor-memory":
         pytest.skip("the 32-bit mode has one route")
     layer, width, eps = MIXERS_ALONE[name], 96, 1e-5
     rng = np.random.RandomState(len(name))
@@ -151,7 +157,7 @@ def test_one_key_that_stands_out(kind, dtype, route):
     """One token's shared key part answers one query direction far above the rest (through the rotation, whatever the distance):
     the asker's result is that token's value.  Spots at the sequence's start, at page borders and tile borders, and hundreds of
     tokens back; asked in a portion, in a portion of two tokens and alone; and the token just behind the asker stays unseen."""
-    if dtype == "float32" and route != "tensor-cores":
+    if dtype == "float32" and route != "tensor-memory":
         pytest.skip("the 32-bit mode has one route")
     H, dk, dr, dv, r, T, width, page = 2, 16, 16, 16, 32, 620, 64, 16
     layer = su.low(H, dk, dr, dv, 48, r, 1.0, 1e9, None) if kind == "low" else su.far(H, dk, dr, dv, r, 1.0, 1e9, (1.0, 64, 32.0, 1.0), None)
@@ -211,7 +217,7 @@ def test_one_key_that_stands_out(kind, dtype, route):
 def test_the_sink_takes_its_share(dtype, route):
     """A sink that drowns a head, one that vanishes and one that weighs as much as a key of score 0, over a portion, a portion of two
     tokens and single tokens (whose keys are shared out over several blocks: the sink counts once)."""
-    if dtype == "float32" and route != "tensor-cores":
+    if dtype == "float32" and route != "tensor-memory":
         pytest.skip("the 32-bit mode has one route")
     layer, width = su.low(3, 16, 16, 32, 32, 64, 0.2, 100.0, None), 96
     rng = np.random.RandomState(5)
