@@ -8,7 +8,7 @@
 // With a sink (one number per head) the softmax's denominator also holds exp(sink_h): it starts the running maximum and
 // mass of the first split's rows.
 //
-// One CTA (8 or 16 warps: 2 or 4 row groups of 4 warps) owns a tile of 32 or 64 query rows, each row one (token, head)
+// One CTA (4, 8 or 16 warps: 1, 2 or 4 row groups of 4 warps) owns a tile of 16, 32 or 64 query rows, each row one (token, head)
 // pair of one request; because every head reads the same keys, a key tile is fetched once for all of them.  Keys stream through shared memory in tiles of 32,
 // gathered page by page with cp.async, two stages deep.  Per key tile:
 //
@@ -31,24 +31,31 @@
 #define LAT_PS 40          // stride of a row of weights (bfloat16)
 #define LAT_LOG2E 1.4426950408889634f
 
+// Where a warp's rows of the tile at key0 are (a warp takes rows warp, warp + warps, ...; lane i looks up its i-th row): the
+// row's number in the pool, negative outside [lo, hi).  One look-up per lane, side by side, a tile ahead of the copies.
+template <int THREADS>
+__device__ __forceinline__ int latent_find_keys(const int32_t* __restrict__ table, int key0, int lo, int hi, int page_size, int page_shift) {
+    constexpr int WARPS = THREADS / 32;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int key = key0 + warp + lane * WARPS;
+    if (lane >= LAT_KEYS / WARPS || key < lo || key >= hi) return -1;
+    const int pidx = page_shift >= 0 ? (key >> page_shift) : (key / page_size);
+    return table[pidx] * page_size + (key - pidx * page_size);
+}
+
 // 32 cache rows [32][WS] (WS = wide rounded up to 16, + 8); rows outside [lo, hi) and the padding are zero
 template <int THREADS>
-__device__ __forceinline__ void latent_load_keys(__nv_bfloat16* dst, const __nv_bfloat16* __restrict__ pool,
-                                                 const int32_t* __restrict__ table, int key0, int lo, int hi, int page_size,
-                                                 int page_shift, int wide, int WS) {
-    // a warp per row (one page lookup per row), a lane per 16-byte piece
+__device__ __forceinline__ void latent_load_keys(__nv_bfloat16* dst, const __nv_bfloat16* __restrict__ pool, int found, int wide, int WS) {
+    // a warp per row, a lane per 16-byte piece
+    constexpr int WARPS = THREADS / 32;
     const int chunks = (WS - 8) / 8, real = wide / 8;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int r = warp; r < LAT_KEYS; r += THREADS / 32) {
-        const int key = key0 + r;
-        const bool ok = key >= lo && key < hi;
-        const __nv_bfloat16* src = pool;
-        if (ok) {
-            const int pidx = page_shift >= 0 ? (key >> page_shift) : (key / page_size);
-            const int slot = key - pidx * page_size;
-            src = pool + ((size_t)table[pidx] * page_size + slot) * wide;
-        }
-        __nv_bfloat16* d = dst + r * WS;
+#pragma unroll
+    for (int i = 0; i < LAT_KEYS / WARPS; ++i) {
+        const int at = __shfl_sync(0xffffffffu, found, i);
+        const bool ok = at >= 0;
+        const __nv_bfloat16* src = pool + (size_t)(ok ? at : 0) * wide;
+        __nv_bfloat16* d = dst + (warp + i * WARPS) * WS;
         for (int part = lane; part < chunks; part += 32) {
             if (ok && part < real) cp_async16(d + part * 8, src + part * 8);
             else *reinterpret_cast<uint4*>(d + part * 8) = make_uint4(0, 0, 0, 0);
@@ -116,9 +123,10 @@ __global__ void __launch_bounds__(RG * 128) attention_latent_kernel(
         }
     }
     const int page_shift = (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;
-    if (kt_begin < kt_end)
-        latent_load_keys<THREADS>(sK, pool, table, kt_begin * LAT_KEYS, lo_all, hi_all, page_size, page_shift, wide, WS);
+    int found = latent_find_keys<THREADS>(table, kt_begin * LAT_KEYS, lo_all, kt_begin < kt_end ? hi_all : 0, page_size, page_shift);
+    if (kt_begin < kt_end) latent_load_keys<THREADS>(sK, pool, found, wide, WS);
     cp_async_commit();
+    found = latent_find_keys<THREADS>(table, (kt_begin + 1) * LAT_KEYS, lo_all, kt_begin + 1 < kt_end ? hi_all : 0, page_size, page_shift);
 
     float o[MT][NT][4];
 #pragma unroll
@@ -140,9 +148,9 @@ __global__ void __launch_bounds__(RG * 128) attention_latent_kernel(
         cp_async_wait<0>();
         __syncthreads();                             // tile kt has landed; everyone is done with tile kt - 1
         if (kt + 1 < kt_end) {
-            latent_load_keys<THREADS>(sK + (buf ^ 1) * LAT_KEYS * WS, pool, table, (kt + 1) * LAT_KEYS, lo_all, hi_all, page_size,
-                             page_shift, wide, WS);
+            latent_load_keys<THREADS>(sK + (buf ^ 1) * LAT_KEYS * WS, pool, found, wide, WS);
             cp_async_commit();
+            found = latent_find_keys<THREADS>(table, (kt + 2) * LAT_KEYS, lo_all, kt + 2 < kt_end ? hi_all : 0, page_size, page_shift);
         }
         const __nv_bfloat16* tK = sK + buf * LAT_KEYS * WS;
         const int key0 = kt * LAT_KEYS;
@@ -297,21 +305,32 @@ __global__ void __launch_bounds__(RG * 128) attention_latent_kernel(
 // out[row] = sum_s w_s o_s / sum_s w_s l_s with w_s = 2^(m_s - max m): the partial results of a row's splits
 __global__ void attention_latent_merge_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ out32, const float* __restrict__ part_o,
                                               const float* __restrict__ part_ml, int rank, int n_splits) {
+    __shared__ float weight[64];                  // of every split (at most 64): 2^(m_s - max m) / mass
     const size_t row = blockIdx.x;
-    const float* ml = part_ml + row * n_splits * 2;
-    float mx = -INFINITY;
-    for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, ml[s * 2]);
-    float mass = 0.0f;
-    for (int s = 0; s < n_splits; ++s) mass += ml[s * 2] == -INFINITY ? 0.0f : exp2f(ml[s * 2] - mx) * ml[s * 2 + 1];
-    const float inv = mass > 0.0f ? 1.0f / mass : 0.0f;
-    for (int col = threadIdx.x; col < rank; col += blockDim.x) {
-        float acc = 0.0f;
+    if (threadIdx.x < 32) {
+        const float2* ml = reinterpret_cast<const float2*>(part_ml) + row * n_splits;
+        const int lane = threadIdx.x;
+        const float2 none = make_float2(-INFINITY, 0.0f);
+        const float2 a = lane < n_splits ? ml[lane] : none, b = lane + 32 < n_splits ? ml[lane + 32] : none;
+        const float mx = warp_max(fmaxf(a.x, b.x));
+        const float wa = a.x == -INFINITY ? 0.0f : exp2f(a.x - mx), wb = b.x == -INFINITY ? 0.0f : exp2f(b.x - mx);
+        const float mass = warp_sum(wa * a.y + wb * b.y);
+        const float inv = mass > 0.0f ? 1.0f / mass : 0.0f;
+        weight[lane] = wa * inv;
+        weight[lane + 32] = wb * inv;
+    }
+    __syncthreads();
+    const float* src = part_o + row * n_splits * rank;
+    for (int col = threadIdx.x * 4; col < rank; col += blockDim.x * 4) {          // rank is a multiple of 16
+        float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
         for (int s = 0; s < n_splits; ++s) {
-            const float m = ml[s * 2];
-            if (m != -INFINITY) acc = fmaf(exp2f(m - mx), part_o[(row * n_splits + s) * rank + col], acc);
+            const float w = weight[s];
+            const float4 v = *reinterpret_cast<const float4*>(src + (size_t)s * rank + col);
+            acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
         }
-        if (out32 != nullptr) out32[row * rank + col] = acc * inv;
-        else out[row * rank + col] = __float2bfloat16(acc * inv);
+        if (out32 != nullptr) *reinterpret_cast<float4*>(out32 + row * rank + col) = acc;
+        else *reinterpret_cast<uint2*>(out + row * rank + col) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
     }
 }
 
@@ -346,7 +365,7 @@ static int launch_latent(LAT_ARGS) {
               scale * LAT_LOG2E, (const float*)sink);
     MM_CHECK_LAUNCH();
     if (n_splits > 1) {
-        mm_launch(attention_latent_merge_kernel, dim3(n_rows), dim3(rank >= 256 ? 128 : 64), 0, s, out_f32 ? nullptr : (__nv_bfloat16*)out,
+        mm_launch(attention_latent_merge_kernel, dim3(n_rows), dim3(rank > 256 ? 128 : (rank > 128 ? 64 : 32)), 0, s, out_f32 ? nullptr : (__nv_bfloat16*)out,
                   out_f32 ? (float*)out : nullptr, (const float*)part_o, (const float*)part_ml, rank, n_splits);
         MM_CHECK_LAUNCH();
     }
@@ -360,18 +379,18 @@ MM_EXPORT int mm_attention_latent_supported(int wide, int rank) {
     return rank >= 16 && rank <= 512 && rank % 16 == 0 && wide >= rank && wide % 8 == 0 && latent_smem(wide, 32) <= LAT_SMEM_MAX;
 }
 
-// the rows of a tile the kernel may be given for this width: 64 (sixteen warps) where that many query rows fit, else 32
+// the most rows of a tile the kernel may be given for this width: 64 (sixteen warps) where that many query rows fit, else 32
 MM_EXPORT int mm_attention_latent_tile_rows(int wide) { return latent_smem(wide, 64) <= LAT_SMEM_MAX ? 64 : 32; }
 
 // q [n, H, wide] and pool [pages, page, wide] bfloat16; out [n, H, rank] bfloat16 or fp32.  tiles int32 [n_tiles, 5] of at
-// most tile_rows (32 or 64) rows each; n_rows = n * H.  n_splits > 1: part_o [n_rows, n_splits, rank] and part_ml
+// most tile_rows (16, 32 or 64) rows each; n_rows = n * H.  n_splits > 1: part_o [n_rows, n_splits, rank] and part_ml
 // [n_rows, n_splits, 2] (fp32).  sink: fp32 [H] or null.
 MM_EXPORT int mm_attention_latent_bf16(const void* q, const void* pool, void* out, void* part_o, void* part_ml, int n_splits,
                                        const void* tiles, int n_tiles, int tile_rows, int n_rows, const void* positions,
                                        const void* table, int table_width, int page_size, int H, int wide, int rank, int window,
                                        float scale, const void* sink, int out_f32, void* stream) {
     MM_REQUIRE(mm_attention_latent_supported(wide, rank), "latent attention: rank a multiple of 16 up to 512, row width a multiple of 8");
-    MM_REQUIRE(tile_rows == 32 || (tile_rows == 64 && mm_attention_latent_tile_rows(wide) == 64), "latent attention: tiles of 32 or 64 rows");
+    MM_REQUIRE(tile_rows == 16 || tile_rows == 32 || (tile_rows == 64 && mm_attention_latent_tile_rows(wide) == 64), "latent attention: tiles of 16, 32 or 64 rows");
     MM_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (part_o != nullptr && part_ml != nullptr)),
                "latent attention: 1..64 splits, with scratch for more than one");
     MM_REQUIRE(n_tiles >= 0 && H > 0 && page_size > 0 && table_width > 0 && window >= 0 && scale > 0.0f,
@@ -383,6 +402,12 @@ MM_EXPORT int mm_attention_latent_bf16(const void* q, const void* pool, void* ou
         if (rank <= 128) return launch_latent<4, 1, 4>(LAT_PASS);
         if (rank <= 256) return launch_latent<8, 1, 4>(LAT_PASS);
         return launch_latent<16, 1, 4>(LAT_PASS);
+    }
+    if (tile_rows == 16) {
+        if (rank <= 64) return launch_latent<2, 1, 1>(LAT_PASS);
+        if (rank <= 128) return launch_latent<4, 1, 1>(LAT_PASS);
+        if (rank <= 256) return launch_latent<8, 1, 1>(LAT_PASS);
+        return launch_latent<16, 1, 1>(LAT_PASS);
     }
     if (rank <= 64) return launch_latent<2, 1, 2>(LAT_PASS);
     if (rank <= 128) return launch_latent<4, 1, 2>(LAT_PASS);

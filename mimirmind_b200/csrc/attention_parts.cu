@@ -9,7 +9,7 @@
 //     the shared rotated key part and every head's rotated query part are turned (pairs i, i + dims/2, or 2i, 2i + 1), and latent and
 //     rotated key are written side by side into one per-token cache array;
 //   * head_matmul: out[t, h, :] = in[t, h, :] . M[h] with a matrix per head (absorbing the key or value up-projection
-//     of a latent attention into the query or the output), fp32 FMAs over eight runs of k, summed in order;
+//     of a latent attention into the query or the output), fp32 FMAs over sixteen runs of k, summed in order;
 //   * head_finish: what happens to each head's attention output before the output projection: the difference of two
 //     maps (a1 - lambda a2), a division by the head's root mean square, a constant factor, a sigmoid gate per (token, head).
 #include "common.cuh"
@@ -106,9 +106,11 @@ template <typename T>
 __global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, int q_off, const float* __restrict__ c_rows, int ldc, int c_off,
                                    const void* __restrict__ norm_w, int w_dtype, float eps, const float2* __restrict__ rot, int rot_dims, int pairs,
                                    T* __restrict__ q_plain, T* __restrict__ q_full, T* __restrict__ pages, const int32_t* __restrict__ slots,
-                                   int page_size, int H, int dk, int dr, int rank, T* __restrict__ q_wide, int wide_rot, int wide_w) {
+                                   int page_size, int H, int dk, int dr, int rank, T* __restrict__ q_wide, int wide_rot, int wide_w, int vec) {
     __shared__ float scratch[32];
     const int t = blockIdx.x;
+    // few tokens: their heads are shared out over gridDim.y blocks, the first of which makes the cached row
+    const int h_lo = H * blockIdx.y / gridDim.y, h_hi = H * (blockIdx.y + 1) / gridDim.y;
     const float* row = q_rows + (size_t)t * ldq;
     const float* crow = c_rows + (size_t)t * ldc;
     const int half = rot_dims / 2;
@@ -117,11 +119,27 @@ __global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, in
     // queries: plain parts to their buffer, rotated parts into the joined query
     if (q_wide != nullptr) {
         const int per = wide_w / 8;
-        for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+        for (int i = h_lo * per + threadIdx.x; i < h_hi * per; i += blockDim.x) {
             const int h = i / per, e0 = (i - h * per) * 8;
             const float* head = row + q_off + h * (dk + dr);
+            const int e = e0 < wide_rot ? e0 : dk + e0 - wide_rot;                 // the piece's place in the head
+            const bool real = e0 < wide_rot ? e0 < dk : e0 - wide_rot < dr;
             __align__(16) T v[8];
-            if (e0 < wide_rot) {
+            if (vec && (!real || e0 < wide_rot || (pairs && e0 - wide_rot + 8 <= rot_dims))) {      // 16-byte reads: a pair never leaves its piece
+                float4 a = make_float4(0.0f, 0.0f, 0.0f, 0.0f), b = a;
+                if (real) {
+                    a = *reinterpret_cast<const float4*>(head + e);
+                    b = *reinterpret_cast<const float4*>(head + e + 4);
+                    if (e0 >= wide_rot) {
+                        const float2* f = rt + (e0 - wide_rot) / 2;
+                        const float2 f0 = f[0], f1 = f[1], f2 = f[2], f3 = f[3];
+                        a = make_float4(a.x * f0.x - a.y * f0.y, a.y * f0.x + a.x * f0.y, a.z * f1.x - a.w * f1.y, a.w * f1.x + a.z * f1.y);
+                        b = make_float4(b.x * f2.x - b.y * f2.y, b.y * f2.x + b.x * f2.y, b.z * f3.x - b.w * f3.y, b.w * f3.x + b.z * f3.y);
+                    }
+                }
+                v[0] = from_f32<T>(a.x); v[1] = from_f32<T>(a.y); v[2] = from_f32<T>(a.z); v[3] = from_f32<T>(a.w);
+                v[4] = from_f32<T>(b.x); v[5] = from_f32<T>(b.y); v[6] = from_f32<T>(b.z); v[7] = from_f32<T>(b.w);
+            } else if (e0 < wide_rot) {
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] = from_f32<T>(e0 < dk ? head[e0 + j] : 0.0f);
             } else {
@@ -133,14 +151,15 @@ __global__ void latent_prep_kernel(const float* __restrict__ q_rows, int ldq, in
             for (int j = 0; j < (int)sizeof(v) / 16; ++j) reinterpret_cast<uint4*>(dst)[j] = reinterpret_cast<const uint4*>(v)[j];
         }
     }
-    for (int i = threadIdx.x; q_plain != nullptr && i < H * dk; i += blockDim.x) {
+    for (int i = h_lo * dk + threadIdx.x; q_plain != nullptr && i < h_hi * dk; i += blockDim.x) {
         const int h = i / dk, e = i - h * dk;
         q_plain[(size_t)t * H * dk + i] = from_f32<T>(row[q_off + h * (dk + dr) + e]);
     }
-    for (int i = threadIdx.x; q_full != nullptr && i < H * dr; i += blockDim.x) {
+    for (int i = h_lo * dr + threadIdx.x; q_full != nullptr && i < h_hi * dr; i += blockDim.x) {
         const int h = i / dr, e = i - h * dr;
         q_full[((size_t)t * H + h) * wide + rank + e] = from_f32<T>(turned(row + q_off + h * (dk + dr) + dk, rt, e, rot_dims, pairs));
     }
+    if (blockIdx.y != 0) return;
     // the latent: divided by its root mean square, times its weight
     float sq = 0.0f;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) sq = fmaf(crow[c_off + i], crow[c_off + i], sq);
@@ -168,14 +187,16 @@ MM_EXPORT int mm_latent_prep(const void* q_rows, int ldq, int q_off, const void*
                                      ((uintptr_t)q_wide & 15) == 0), "latent prep: wide queries need parts of multiples of 8 that fit their places");
     if (n_tokens == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
+    const dim3 grid(n_tokens, n_tokens <= 64 ? (H < 8 ? H : 8) : 1);
+    const int vec = ldq % 4 == 0 && q_off % 4 == 0 && ((uintptr_t)q_rows & 15) == 0;
     if (dtype == MM_F32)
-        mm_launch(latent_prep_kernel<float>, dim3(n_tokens), dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
+        mm_launch(latent_prep_kernel<float>, grid, dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
                   norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (float*)q_plain, (float*)q_full, (float*)pages, (const int32_t*)slots, page_size, H, dk, dr, rank,
-                  (float*)q_wide, wide_rot, wide_w);
+                  (float*)q_wide, wide_rot, wide_w, vec);
     else if (dtype == MM_BF16)
-        mm_launch(latent_prep_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
+        mm_launch(latent_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, (const float*)q_rows, ldq, q_off, (const float*)c_rows, ldc, c_off,
                   norm_w, w_dtype, eps, (const float2*)rot, rot_dims, pairs, (__nv_bfloat16*)q_plain, (__nv_bfloat16*)q_full, (__nv_bfloat16*)pages, (const int32_t*)slots,
-                  page_size, H, dk, dr, rank, (__nv_bfloat16*)q_wide, wide_rot, wide_w);
+                  page_size, H, dk, dr, rank, (__nv_bfloat16*)q_wide, wide_rot, wide_w, vec);
     else
         MM_REQUIRE(false, "latent prep: dtype must be float32 or bfloat16");
     MM_CHECK_LAUNCH();
@@ -186,20 +207,40 @@ MM_EXPORT int mm_latent_prep(const void* q_rows, int ldq, int q_off, const void*
 // out[t, h, j] = sum_k in[t, h, k] M[h, k, j]; in: token stride in_ld, head stride in_hs; out likewise.  Eight tokens
 // of one head per block share each matrix element; a thread owns one output column.
 #define HM_TOKENS 8
-#define HM_COLS 64
-#define HM_SLICES 8
+#define HM_COLS 32
+#define HM_SLICES 16
+#define HM_AHEAD 16
 // A block of HM_COLS x HM_SLICES threads makes HM_TOKENS tokens x HM_COLS columns of one head: slice y sums its run of k
 // (ascending), then thread (x, y) adds the slices' sums of token y in slice order.  The cut of k depends on K alone, so
 // a token's result never depends on the batch.
 template <typename T>
 __global__ void __launch_bounds__(HM_COLS * HM_SLICES) head_matmul_kernel(
     const T* __restrict__ in, long long in_ld, int in_hs, const T* __restrict__ M, T* __restrict__ out, long long out_ld, int out_hs,
-    int n_tokens, int K, int N) {
+    int n_tokens, int K, int N, int vec) {
     extern __shared__ float in_s[];   // [HM_TOKENS][K]
     __shared__ float part[HM_SLICES][HM_TOKENS][HM_COLS];
     const int h = blockIdx.y, t0 = blockIdx.z * HM_TOKENS;
     const int x = threadIdx.x, y = threadIdx.y, tid = y * HM_COLS + x;
     const int j = blockIdx.x * HM_COLS + x;
+    const int per = (K + HM_SLICES - 1) / HM_SLICES;
+    const int k_lo = y * per, k_hi = min(K, k_lo + per);
+    const T* Mh = M + (size_t)h * K * N + j;
+    // the first matrix elements need nobody else: they are under way while the rows are staged
+    T first[HM_AHEAD];
+#pragma unroll
+    for (int u = 0; u < HM_AHEAD; ++u) first[u] = (j < N && k_lo + u < k_hi) ? Mh[(size_t)(k_lo + u) * N] : from_f32<T>(0.0f);
+    if (vec) {                                    // rows of 16-byte words
+        constexpr int W = 16 / (int)sizeof(T);
+        const int words = K / W;
+        for (int i = tid; i < HM_TOKENS * words; i += HM_COLS * HM_SLICES) {
+            const int tt = i / words, k = (i - tt * words) * W;
+            uint4 raw = make_uint4(0, 0, 0, 0);
+            if (t0 + tt < n_tokens) raw = *reinterpret_cast<const uint4*>(in + (size_t)(t0 + tt) * in_ld + (size_t)h * in_hs + k);
+            const T* v = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+            for (int u = 0; u < W; ++u) in_s[tt * K + k + u] = to_f32<T>(v[u]);
+        }
+    } else
     for (int i = tid; i < HM_TOKENS * K; i += HM_COLS * HM_SLICES) {
         const int tt = i / K, k = i - tt * K;
         in_s[i] = (t0 + tt < n_tokens) ? to_f32<T>(in[(size_t)(t0 + tt) * in_ld + (size_t)h * in_hs + k]) : 0.0f;
@@ -208,12 +249,17 @@ __global__ void __launch_bounds__(HM_COLS * HM_SLICES) head_matmul_kernel(
     float acc[HM_TOKENS];
 #pragma unroll
     for (int tt = 0; tt < HM_TOKENS; ++tt) acc[tt] = 0.0f;
-    const int per = (K + HM_SLICES - 1) / HM_SLICES;
-    const int k_lo = y * per, k_hi = min(K, k_lo + per);
     if (j < N) {
-        const T* Mh = M + (size_t)h * K * N + j;
-#pragma unroll 4
-        for (int k = k_lo; k < k_hi; ++k) {
+#pragma unroll
+        for (int u = 0; u < HM_AHEAD; ++u) {
+            if (k_lo + u < k_hi) {
+                const float w = to_f32<T>(first[u]);
+#pragma unroll
+                for (int tt = 0; tt < HM_TOKENS; ++tt) acc[tt] = fmaf(in_s[tt * K + k_lo + u], w, acc[tt]);
+            }
+        }
+#pragma unroll 16
+        for (int k = k_lo + HM_AHEAD; k < k_hi; ++k) {
             const float w = to_f32<T>(Mh[(size_t)k * N]);
 #pragma unroll
             for (int tt = 0; tt < HM_TOKENS; ++tt) acc[tt] = fmaf(in_s[tt * K + k], w, acc[tt]);
@@ -222,7 +268,7 @@ __global__ void __launch_bounds__(HM_COLS * HM_SLICES) head_matmul_kernel(
 #pragma unroll
     for (int tt = 0; tt < HM_TOKENS; ++tt) part[y][tt][x] = acc[tt];
     __syncthreads();
-    if (j >= N || t0 + y >= n_tokens) return;
+    if (y >= HM_TOKENS || j >= N || t0 + y >= n_tokens) return;
     float sum = 0.0f;
 #pragma unroll
     for (int sl = 0; sl < HM_SLICES; ++sl) sum += part[sl][y][x];
@@ -237,6 +283,8 @@ MM_EXPORT int mm_head_matmul(const void* in, long long in_ld, int in_hs, const v
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)HM_TOKENS * K * sizeof(float);
     const dim3 grid(ceil_div(N, HM_COLS), H, ceil_div(n_tokens, HM_TOKENS)), block(HM_COLS, HM_SLICES);
+    const int w = dtype == MM_F32 ? 4 : 8;         // numbers of a 16-byte word
+    const int vec = K % w == 0 && in_ld % w == 0 && in_hs % w == 0 && ((uintptr_t)in & 15) == 0;
     if (grid.z > 65535) {
         mm_set_last_error("head product: too many tokens for one launch");
         return MM_ERR_BAD_ARG;
@@ -244,11 +292,11 @@ MM_EXPORT int mm_head_matmul(const void* in, long long in_ld, int in_hs, const v
     if (dtype == MM_F32) {
         if (smem > 32 * 1024) cudaFuncSetAttribute(head_matmul_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         mm_launch(head_matmul_kernel<float>, grid, block, smem, s, (const float*)in, in_ld, in_hs, (const float*)M, (float*)out, out_ld, out_hs,
-                  n_tokens, K, N);
+                  n_tokens, K, N, vec);
     } else if (dtype == MM_BF16) {
         if (smem > 32 * 1024) cudaFuncSetAttribute(head_matmul_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         mm_launch(head_matmul_kernel<__nv_bfloat16>, grid, block, smem, s, (const __nv_bfloat16*)in, in_ld, in_hs, (const __nv_bfloat16*)M,
-                  (__nv_bfloat16*)out, out_ld, out_hs, n_tokens, K, N);
+                  (__nv_bfloat16*)out, out_ld, out_hs, n_tokens, K, N, vec);
     } else {
         MM_REQUIRE(false, "head product: dtype must be float32 or bfloat16");
     }

@@ -651,10 +651,26 @@ __global__ void gather_rows_kernel(const T* __restrict__ src, const int32_t* __r
     for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = s[i];
 }
 
+// rows of `words` 16-byte words: a warp per row, four words in flight per lane
+__global__ void gather_rows16_kernel(const uint4* __restrict__ src, const int32_t* __restrict__ rows, uint4* __restrict__ out, int n_rows, int words) {
+    const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (row >= n_rows) return;
+    const uint4* s = src + (size_t)rows[row] * words;
+    uint4* o = out + (size_t)row * words;
+#pragma unroll 4
+    for (int i = threadIdx.x & 31; i < words; i += 32) o[i] = s[i];
+}
+
 MM_EXPORT int mm_gather_rows(const void* src, const void* rows, void* out, int dtype, int n_rows, int d, void* stream) {
     MM_REQUIRE(n_rows >= 0 && d > 0, "gather_rows: bad sizes");
     if (n_rows == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
+    const long long bytes = (long long)d * (dtype == MM_F32 ? 4 : 2);
+    if ((dtype == MM_F32 || dtype == MM_BF16) && bytes % 16 == 0 && (((uintptr_t)src | (uintptr_t)out) & 15) == 0) {
+        gather_rows16_kernel<<<ceil_div(n_rows, 4), 128, 0, s>>>((const uint4*)src, (const int32_t*)rows, (uint4*)out, n_rows, (int)(bytes / 16));
+        MM_CHECK_LAUNCH();
+        return MM_OK;
+    }
     if (dtype == MM_F32) gather_rows_kernel<float><<<n_rows, 256, 0, s>>>((const float*)src, (const int32_t*)rows, (float*)out, d);
     else if (dtype == MM_BF16) gather_rows_kernel<__nv_bfloat16><<<n_rows, 256, 0, s>>>((const __nv_bfloat16*)src, (const int32_t*)rows, (__nv_bfloat16*)out, d);
     else MM_REQUIRE(false, "gather_rows: dtype must be float32 or bfloat16");

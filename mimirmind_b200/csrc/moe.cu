@@ -128,8 +128,9 @@ __global__ void moe_route_kernel(const float* __restrict__ z, int ldz, int n_tok
     moe_route_warp(z + (size_t)t * ldz, s, lane, E, top, groups, keep, idx, wts, (size_t)t, scoring);
 }
 
-// The router's product and its choice in one launch, one block per token: every warp takes experts in turn and sums
-// x . w_e over lanes in fp32 (a fixed order, whatever else is in the batch); then the first warp chooses.
+// The router's product and its choice in one launch, TOK tokens per block: every warp takes experts in turn and sums
+// x . w_e over lanes in fp32 (a fixed order, whatever else is in the batch and however many tokens share a block's reads of w);
+// then one warp per token chooses.
 template <typename T>
 __device__ __forceinline__ void load8(const T* p, float* v);
 template <>
@@ -149,41 +150,62 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
     }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) moe_router_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, int D, int E, int top,
+template <typename T, int TOK>
+__global__ void __launch_bounds__(1024) moe_router_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, int n_tokens, int D, int E, int top,
                                                          int groups, int keep, int vec, int32_t* __restrict__ idx, float* __restrict__ wts, int scoring,
                                                          const float* __restrict__ correction, int pair_sum, float* __restrict__ gate) {
-    extern __shared__ float route_smem[];      // logits [E + 1], then the choice's scratch
+    extern __shared__ float route_smem[];      // per token: logits [E + 1], then the choice's scratch [2 E + 2 groups]
     const int rows = gate ? E + 1 : E;         // with a gate the matrix has one more row, for it
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const size_t t = blockIdx.x;
-    const T* xr = x + t * ldx;
-    for (int e = warp; e < rows; e += 8) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int per_token = 3 * E + 1 + 2 * groups;
+    const size_t t0 = (size_t)blockIdx.x * TOK;
+    const T* xr[TOK];
+#pragma unroll
+    for (int k = 0; k < TOK; ++k) xr[k] = x + min(t0 + k, (size_t)n_tokens - 1) * ldx;
+    for (int e = warp; e < rows; e += warps) {
         const float* we = w + (size_t)e * D;
-        float acc = 0.0f;
+        float acc[TOK], a2[TOK];
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) acc[k] = a2[k] = 0.0f;
         if (vec) {        // rows that start on 16-byte boundaries: eight numbers per lane and step, several steps in flight
-            float a2 = 0.0f;
-#pragma unroll 4
+#pragma unroll (TOK == 1 ? 8 : 2)
             for (int d = lane * 8; d < D; d += 256) {
-                float xv[8], wv[8];
-                load8<T>(xr + d, xv);
+                float wv[8];
                 load8<float>(we + d, wv);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    acc = fmaf(xv[i], wv[i], acc);
-                    a2 = fmaf(xv[4 + i], wv[4 + i], a2);
+                for (int k = 0; k < TOK; ++k) {
+                    float xv[8];
+                    load8<T>(xr[k] + d, xv);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        acc[k] = fmaf(xv[i], wv[i], acc[k]);
+                        a2[k] = fmaf(xv[4 + i], wv[4 + i], a2[k]);
+                    }
                 }
             }
-            acc += a2;
+#pragma unroll
+            for (int k = 0; k < TOK; ++k) acc[k] += a2[k];
         } else {
-            for (int d = lane; d < D; d += 32) acc = fmaf(to_f32<T>(xr[d]), we[d], acc);
+            for (int d = lane; d < D; d += 32) {
+                const float wd = we[d];
+#pragma unroll
+                for (int k = 0; k < TOK; ++k) acc[k] = fmaf(to_f32<T>(xr[k][d]), wd, acc[k]);
+            }
         }
-        acc = warp_sum(acc);
-        if (lane == 0) route_smem[e] = acc;
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+            const float z = warp_sum(acc[k]);
+            if (lane == 0) route_smem[k * per_token + e] = z;
+        }
     }
     __syncthreads();
-    if (gate && threadIdx.x == 32) gate[t] = 1.0f / (1.0f + expf(-route_smem[E]));
-    if (warp == 0) moe_route_warp(route_smem, route_smem + E + 1, lane, E, top, groups, keep, idx, wts, t, scoring, correction, pair_sum);
+    for (int k = warp; k < TOK; k += warps) {
+        const size_t t = t0 + k;
+        if (t >= (size_t)n_tokens) break;
+        float* mine = route_smem + k * per_token;
+        if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-mine[E]));
+        moe_route_warp(mine, mine + E + 1, lane, E, top, groups, keep, idx, wts, t, scoring, correction, pair_sum);
+    }
 }
 
 // w fp32 [E, D], or [E + 1, D] with `gate` (fp32 [n_tokens]), which gets the logistic of the last row's product;
@@ -193,16 +215,23 @@ MM_EXPORT int mm_moe_router_choice(const void* x, int x_dtype, int ldx, const vo
     MM_REQUIRE(scoring == 0 || scoring == 1, "moe router: the scoring is 0 (softmax, renormed) or 1 (sigmoid, as it is)");
     MM_REQUIRE(n_tokens >= 0 && D > 0 && ldx >= D && E > 0 && top > 0 && top <= E && groups > 0 && E % groups == 0 && keep > 0 && keep <= groups,
                "moe router: experts must split into equal runs, and 0 < top <= experts, 0 < keep <= runs");
-    const size_t smem = (size_t)(3 * E + 1 + 2 * groups) * sizeof(float);
-    MM_REQUIRE(smem <= 48 * 1024, "moe router: too many experts for the router's shared memory");
+    const size_t per_token = (size_t)(3 * E + 1 + 2 * groups) * sizeof(float);
+    MM_REQUIRE(per_token <= 48 * 1024, "moe router: too many experts for the router's shared memory");
     if (n_tokens == 0) return MM_OK;
+    // many tokens: four share a block, which then reads the matrix a quarter as often; few: a warp per expert
+    const int tok = n_tokens >= 512 && 4 * per_token <= 48 * 1024 ? 4 : 1;
+    const int rows = gate ? E + 1 : E;
+    const int threads = tok == 4 ? 256 : 32 * (rows < 8 ? 8 : (rows < 32 ? rows : 32));
+    const size_t smem = per_token * tok;
+    const dim3 blocks(ceil_div(n_tokens, tok));
     const int vec = D % 8 == 0 && ldx % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
     if (x_dtype == MM_F32)
-        mm_launch(moe_router_kernel<float>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, (const float*)x, ldx, (const float*)w, D, E, top,
-                  groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate);
+        mm_launch(tok == 4 ? moe_router_kernel<float, 4> : moe_router_kernel<float, 1>, blocks, dim3(threads), smem, (cudaStream_t)stream, (const float*)x, ldx,
+                  (const float*)w, n_tokens, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate);
     else if (x_dtype == MM_BF16)
-        mm_launch(moe_router_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, (const __nv_bfloat16*)x, ldx,
-                  (const float*)w, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate);
+        mm_launch(tok == 4 ? moe_router_kernel<__nv_bfloat16, 4> : moe_router_kernel<__nv_bfloat16, 1>, blocks, dim3(threads), smem, (cudaStream_t)stream,
+                  (const __nv_bfloat16*)x, ldx, (const float*)w, n_tokens, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring,
+                  (const float*)correction, pair_sum, (float*)gate);
     else
         MM_REQUIRE(false, "moe router: dtype must be float32 or bfloat16");
     MM_CHECK_LAUNCH();
@@ -352,30 +381,40 @@ MM_EXPORT int mm_moe_sort(const void* idx, int n_rows, int E, void* offsets, voi
 // ---------------------------------------------------------------------------------------------------------------
 // the experts' products over their rows
 // ---------------------------------------------------------------------------------------------------------------
-// A CTA's tile: expert e and rows [lo, hi) of the sorted order, found from the offsets (every expert's rows start a
-// tile of their own).  Returns false when the CTA has no tile.
+// A CTA's tile: expert and rows [lo, hi) of the sorted order, found from the offsets (every expert's rows start a tile of
+// their own) by one warp, 32 experts at a time; info = (expert, lo, hi), expert -1 when the CTA has no tile.
 template <int TM>
-__device__ __forceinline__ bool moe_tile(const int32_t* __restrict__ offsets, int E, int tile, int& e, int& lo, int& hi) {
+__device__ __forceinline__ void moe_tile(const int32_t* __restrict__ offsets, int E, int tile, int lane, int* info) {
     int seen = 0;
-    for (int x = 0; x < E; ++x) {
-        const int a = offsets[x], b = offsets[x + 1];
+    if (lane == 0) info[0] = -1;
+    __syncwarp();
+    for (int base = 0; base < E; base += 32) {
+        const int x = base + lane;
+        const int a = x < E ? offsets[x] : 0, b = x < E ? offsets[x + 1] : 0;
         const int tiles = (b - a + TM - 1) / TM;
-        if (tile < seen + tiles) {
-            e = x;
-            lo = a + (tile - seen) * TM;
-            hi = min(lo + TM, b);
-            return true;
+        int upto = tiles;                       // tiles of the experts up to this lane's
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int v = __shfl_up_sync(0xffffffffu, upto, o);
+            if (lane >= o) upto += v;
         }
-        seen += tiles;
+        const int first = seen + upto - tiles;
+        if (tile >= first && tile < first + tiles) {
+            info[0] = x;
+            info[1] = a + (tile - first) * TM;
+            info[2] = min(info[1] + TM, b);
+        }
+        seen += __shfl_sync(0xffffffffu, upto, 31);
+        if (tile < seen) break;
     }
-    return false;
 }
 
 #define MOE_BM 64
 #define MOE_BN 64
 #define MOE_BK 16
 #define MOE_MMA_BK 64
-#define MOE_STAGES 3
+#define MOE_SMALL_BM 16
+__host__ __device__ constexpr int moe_stages(int bm, bool gated) { return bm == 64 ? 3 : (gated ? 3 : 4); }
 
 // What a product of the experts reads and writes.  GATED: W is [E, 2F, K], the gate's rows then the up rows, and the output
 // is act(gate) * up over F columns, the input rows gathered through order / top; SINGLE: W is [E, F, K], the output act(up), the input
@@ -394,13 +433,7 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const TA* __restrict
     __shared__ int32_t rows[MOE_BM];
     __shared__ int tile_info[3];
     const int tid = threadIdx.x;
-    if (tid == 0) {
-        int e = -1, lo = 0, hi = 0;
-        if (!moe_tile<MOE_BM>(offsets, E, blockIdx.y, e, lo, hi)) e = -1;
-        tile_info[0] = e;
-        tile_info[1] = lo;
-        tile_info[2] = hi;
-    }
+    if (tid < 32) moe_tile<MOE_BM>(offsets, E, blockIdx.y, tid, tile_info);
     __syncthreads();
     const int e = tile_info[0], lo = tile_info[1], hi = tile_info[2];
     if (e < 0) return;
@@ -474,50 +507,46 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const TA* __restrict
     }
 }
 
-// bfloat16 on the tensor cores (mma.sync m16n8k16, fp32 accumulation): the same tiles, 64 rows x 64 columns, four
-// warps of 32 x 32 (gated: gate and up accumulators side by side), K in steps of 64 through a ring of shared-memory stages.
-template <int MODE, typename TC>
+// bfloat16 on the tensor cores (mma.sync m16n8k16, fp32 accumulation), K in steps of 64 through a ring of shared-memory stages:
+// tiles of 64 rows x 64 columns, four warps of 32 x 32 (gated: gate and up accumulators side by side), or, where no expert can have
+// more than 16 rows (a decode step), of 16 rows x 64 columns, four warps of 16 x 16, with as many stages as let a whole decode step's CTAs be resident at once.
+template <int MODE, typename TC, int BM>
 __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W,
                                                            TC* __restrict__ C, int ldc, const int32_t* __restrict__ offsets,
                                                            const int32_t* __restrict__ order, int E, int top, int N, int K, int interleaved, int act, float limit,
                                                            const float* __restrict__ row_scale) {
-    // K in steps of 64 through a ring of MOE_STAGES stages: a decode step's tiles hold a handful of rows and stream a
+    // K in steps of 64 through a ring of stages: a decode step's tiles hold a handful of rows and stream a
     // whole expert, so what counts is how many bytes of weights a CTA keeps in flight (rows of 144 bytes: ldmatrix
     // reads without bank conflicts)
     constexpr bool GATED = MODE == MOE_GATED, GATHER = MODE != MOE_DOWN;
     constexpr int BK = MOE_MMA_BK, LD = BK + 8;
     constexpr int WROWS_ = GATED ? 2 * MOE_BN : MOE_BN;
+    constexpr int MI = BM == 64 ? 2 : 1, NCOLS = BM == 64 ? 32 : 16, NJ = NCOLS / 16, STAGES = moe_stages(BM, GATED);
     extern __shared__ __align__(16) unsigned char moe_smem[];
-    typedef __nv_bfloat16 (*ATile)[MOE_BM][LD];
+    typedef __nv_bfloat16 (*ATile)[BM][LD];
     typedef __nv_bfloat16 (*WTile)[WROWS_][LD];
     ATile As = reinterpret_cast<ATile>(moe_smem);
-    WTile Ws = reinterpret_cast<WTile>(moe_smem + sizeof(__nv_bfloat16) * MOE_STAGES * MOE_BM * LD);
-    __shared__ int32_t rows[MOE_BM];
+    WTile Ws = reinterpret_cast<WTile>(moe_smem + sizeof(__nv_bfloat16) * STAGES * BM * LD);
+    __shared__ int32_t rows[BM];
     __shared__ int tile_info[3];
     const int tid = threadIdx.x;
-    if (tid == 0) {
-        int e = -1, lo = 0, hi = 0;
-        if (!moe_tile<MOE_BM>(offsets, E, blockIdx.y, e, lo, hi)) e = -1;
-        tile_info[0] = e;
-        tile_info[1] = lo;
-        tile_info[2] = hi;
-    }
+    if (tid < 32) moe_tile<BM>(offsets, E, blockIdx.y, tid, tile_info);
     __syncthreads();
     const int e = tile_info[0], lo = tile_info[1], hi = tile_info[2];
     if (e < 0) return;
     const int M = hi - lo;
-    if (tid < MOE_BM) rows[tid] = tid < M ? (GATHER ? order[lo + tid] / top : lo + tid) : -1;
+    if (tid < BM) rows[tid] = tid < M ? (GATHER ? order[lo + tid] / top : lo + tid) : -1;
     __syncthreads();
     const int warp = tid >> 5, lane = tid & 31;
-    const int wm = (warp >> 1) * 32, wn = (warp & 1) * 32;
+    const int wm = BM == 64 ? (warp >> 1) * 32 : 0, wn = BM == 64 ? (warp & 1) * 32 : warp * 16;
     const int n0 = blockIdx.x * MOE_BN;
     const __nv_bfloat16* We = W + (size_t)e * (GATED ? 2 : 1) * N * K;
     constexpr int WROWS = GATED ? 2 * MOE_BN : MOE_BN;
-    float acc[2][4][4], up[GATED ? 2 : 1][4][4];
+    float acc[MI][2 * NJ][4], up[GATED ? MI : 1][2 * NJ][4];
 #pragma unroll
-    for (int a = 0; a < 2; ++a)
+    for (int a = 0; a < MI; ++a)
 #pragma unroll
-        for (int b = 0; b < 4; ++b)
+        for (int b = 0; b < 2 * NJ; ++b)
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
                 acc[a][b][c] = 0.0f;
@@ -525,7 +554,7 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
             }
     auto load = [&](int stage, int k0) {
         // 16-byte chunks: 8 per row of 64 k
-        for (int i = tid; i < MOE_BM * 8; i += 128) {
+        for (int i = tid; i < BM * 8; i += 128) {
             const int r = i >> 3, c = (i & 7) * 8;
             __nv_bfloat16* dst = &As[stage][r][c];
             if (rows[r] >= 0 && k0 + c < K) cp_async16(dst, A + (size_t)rows[r] * lda + k0 + c);
@@ -546,36 +575,36 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
     };
     const int steps = (K + BK - 1) / BK;
 #pragma unroll
-    for (int p = 0; p < MOE_STAGES - 1; ++p) {
+    for (int p = 0; p < STAGES - 1; ++p) {
         if (p < steps) load(p, p * BK);
         else cp_async_commit();              // an empty group keeps the count of groups in step
     }
     for (int s = 0; s < steps; ++s) {
-        cp_async_wait<MOE_STAGES - 2>();     // the copies of step s have landed
+        cp_async_wait<STAGES - 2>();     // the copies of step s have landed
         __syncthreads();                     // ... for every thread, and the stage of step s - 1 is free
-        if (s + MOE_STAGES - 1 < steps) load((s + MOE_STAGES - 1) % MOE_STAGES, (s + MOE_STAGES - 1) * BK);
+        if (s + STAGES - 1 < steps) load((s + STAGES - 1) % STAGES, (s + STAGES - 1) * BK);
         else cp_async_commit();
-        const int st = s % MOE_STAGES;
+        const int st = s % STAGES;
 #pragma unroll
         for (int kk = 0; kk < BK; kk += 16) {
-            uint32_t af[2][4];
+            uint32_t af[MI][4];
 #pragma unroll
-            for (int mi = 0; mi < 2; ++mi)
+            for (int mi = 0; mi < MI; ++mi)
                 ldmatrix_x4(af[mi][0], af[mi][1], af[mi][2], af[mi][3], &As[st][wm + mi * 16 + (lane & 15)][kk + (lane >> 4) * 8]);
 #pragma unroll
-            for (int nj = 0; nj < 2; ++nj) {
+            for (int nj = 0; nj < NJ; ++nj) {
                 uint32_t b0, b1, b2, b3;
                 // rows wn + nj*16 .. +15 of W: matrices (n 0-7, k 0-7), (n 0-7, k 8-15), (n 8-15, k 0-7), (n 8-15, k 8-15)
                 ldmatrix_x4(b0, b1, b2, b3, &Ws[st][wn + nj * 16 + (lane & 7) + ((lane >> 4) << 3)][kk + ((lane >> 3) & 1) * 8]);
 #pragma unroll
-                for (int mi = 0; mi < 2; ++mi) {
+                for (int mi = 0; mi < MI; ++mi) {
                     mma_bf16(acc[mi][nj * 2], af[mi], b0, b1);
                     mma_bf16(acc[mi][nj * 2 + 1], af[mi], b2, b3);
                 }
                 if (GATED) {
                     ldmatrix_x4(b0, b1, b2, b3, &Ws[st][MOE_BN + wn + nj * 16 + (lane & 7) + ((lane >> 4) << 3)][kk + ((lane >> 3) & 1) * 8]);
 #pragma unroll
-                    for (int mi = 0; mi < 2; ++mi) {
+                    for (int mi = 0; mi < MI; ++mi) {
                         mma_bf16(up[mi][nj * 2], af[mi], b0, b1);
                         mma_bf16(up[mi][nj * 2 + 1], af[mi], b2, b3);
                     }
@@ -584,14 +613,14 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const __nv_bfloat16* 
         }
     }
 #pragma unroll
-    for (int mi = 0; mi < 2; ++mi)
+    for (int mi = 0; mi < MI; ++mi)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const int m = wm + mi * 16 + (lane >> 2) + half * 8;
             if (m >= M) continue;
             const size_t out_row = GATHER ? (size_t)(lo + m) : (size_t)order[lo + m];
 #pragma unroll
-            for (int ni = 0; ni < 4; ++ni)
+            for (int ni = 0; ni < 2 * NJ; ++ni)
 #pragma unroll
                 for (int c = 0; c < 2; ++c) {
                     const int n = n0 + wn + ni * 8 + (lane & 3) * 2 + c;
@@ -624,25 +653,30 @@ MM_EXPORT int mm_moe_gemm_act(const void* A, int a_dtype, int lda, const void* W
     const int32_t* off = (const int32_t*)offsets;
     const int32_t* ord = (const int32_t*)order;
     if (tensor_cores && a_dtype == MM_BF16 && w_dtype == MM_BF16 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
-        const size_t tile_smem = sizeof(bf) * MOE_STAGES * (MOE_BM + (gated == 1 ? 2 : 1) * MOE_BN) * (MOE_MMA_BK + 8);
-        static bool configured = false;
-        if (!configured) {
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_GATED, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + 2 * MOE_BN) * (MOE_MMA_BK + 8)));
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_SINGLE, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_DOWN, bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
-            cudaFuncSetAttribute(moe_gemm_mma_kernel<MOE_DOWN, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(sizeof(bf) * MOE_STAGES * (MOE_BM + MOE_BN) * (MOE_MMA_BK + 8)));
-            configured = true;
-        }
-        if (gated == 2 && c_dtype == MM_BF16)
-            mm_launch(moe_gemm_mma_kernel<MOE_SINGLE, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, 0, act, limit, row_scale);
-        else if (gated && c_dtype == MM_BF16)
-            mm_launch(moe_gemm_mma_kernel<MOE_GATED, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, interleaved, act, limit, row_scale);
-        else if (!gated && c_dtype == MM_BF16)
-            mm_launch(moe_gemm_mma_kernel<MOE_DOWN, bf>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (bf*)C, ldc, off, ord, E, top, N, K, 0, 0, 0.0f, (const float*)nullptr);
-        else if (!gated && c_dtype == MM_F32)
-            mm_launch(moe_gemm_mma_kernel<MOE_DOWN, float>, grid, dim3(128), tile_smem, s, (const bf*)A, lda, (const bf*)W, (float*)C, ldc, off, ord, E, top, N, K, 0, 0, 0.0f, (const float*)nullptr);
+        // a token chooses an expert once: with at most 16 tokens no expert has more than 16 rows
+        const bool small = n_rows <= MOE_SMALL_BM * top;
+#define MOE_MMA(MODE, TC)                                                                                                                     \
+    do {                                                                                                                                      \
+        constexpr bool G = MODE == MOE_GATED;                                                                                                 \
+        constexpr int smem64 = (int)(sizeof(bf) * moe_stages(64, G) * (64 + (G ? 2 : 1) * MOE_BN) * (MOE_MMA_BK + 8));                         \
+        constexpr int smem16 = (int)(sizeof(bf) * moe_stages(16, G) * (16 + (G ? 2 : 1) * MOE_BN) * (MOE_MMA_BK + 8));                         \
+        static bool configured = false;                                                                                                       \
+        if (!configured) {                                                                                                                    \
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<MODE, TC, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem64);                      \
+            cudaFuncSetAttribute(moe_gemm_mma_kernel<MODE, TC, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem16);                      \
+            configured = true;                                                                                                                \
+        }                                                                                                                                     \
+        mm_launch(small ? moe_gemm_mma_kernel<MODE, TC, 16> : moe_gemm_mma_kernel<MODE, TC, 64>,                                               \
+                  small ? dim3(grid.x, E < n_rows ? E : n_rows) : grid, dim3(128), (size_t)(small ? smem16 : smem64), s, (const bf*)A, lda, (const bf*)W, (TC*)C, ldc, off, ord, \
+                  E, top, N, K, interleaved, act, limit, row_scale);                                                                          \
+    } while (0)
+        if (gated == 2 && c_dtype == MM_BF16) MOE_MMA(MOE_SINGLE, bf);
+        else if (gated == 1 && c_dtype == MM_BF16) MOE_MMA(MOE_GATED, bf);
+        else if (!gated && c_dtype == MM_BF16) MOE_MMA(MOE_DOWN, bf);
+        else if (!gated && c_dtype == MM_F32) MOE_MMA(MOE_DOWN, float);
         else
             MM_REQUIRE(false, "moe gemm: this combination of dtypes is not built");
+#undef MOE_MMA
         MM_CHECK_LAUNCH();
         return MM_OK;
     }

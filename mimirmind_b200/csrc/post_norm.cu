@@ -267,9 +267,22 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, TO* __restrict__ o
     if (i < total) out[i] = from_f32<TO>(x[i]);
 }
 
+__global__ void cast_rows8_kernel(const float* __restrict__ x, __nv_bfloat16* __restrict__ out, long long total8) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total8) return;
+    float v[8];
+    pn_load8(x + i * 8, v);
+    pn_store8(out + i * 8, v);
+}
+
 MM_EXPORT int mm_cast_rows(const void* x, void* out, int out_dtype, long long total, void* stream) {
     MM_REQUIRE(total >= 0, "cast: bad size");
     if (total == 0) return MM_OK;
+    if (out_dtype == MM_BF16 && total % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0) {
+        mm_launch(cast_rows8_kernel, dim3(ceil_div(total / 8, 256)), dim3(256), 0, (cudaStream_t)stream, (const float*)x, (__nv_bfloat16*)out, total / 8);
+        MM_CHECK_LAUNCH();
+        return MM_OK;
+    }
     const dim3 grid(ceil_div(total, 256));
     if (out_dtype == MM_F32)
         mm_launch(cast_rows_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, (const float*)x, (float*)out, total);

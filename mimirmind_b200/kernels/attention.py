@@ -181,6 +181,9 @@ def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, 
 
 USE_LATENT_MMA = True      # False: the latent attention always runs the fp32-arithmetic kernel (tests compare the two)
 LATENT_TILE_ROWS = 32
+LATENT_SMALL_TILE_ROWS = 16
+LATENT_SPLIT_KEYS = 64     # keys per split at least
+LATENT_MAX_SPLITS = 64     # what the kernel takes
 USE_LATENT_WIDE_TILES = True    # False: tiles of 32 rows also for portions of prompts (tests run both)
 LATENT_KEYS = 32
 _latent_declared = False
@@ -197,6 +200,12 @@ def _latent_lib():
         _lib.declare("mm_attention_latent_bf16", [P, P, P, P, P, I, P, I, I, I, P, P, I, I, I, I, I, I, F, P, I, P])
         _latent_declared = True
     return _lib.load()
+
+
+def latent_tile_bytes(wide: int, tile_rows: int) -> int:
+    """Shared memory of a CTA of the tensor-core kernel: queries, two key tiles, partial scores, weights."""
+    row = 2 * (-(-wide // 16) * 16 + 8)
+    return (tile_rows + 2 * LATENT_KEYS) * row + tile_rows * (4 * 33 * 4 + 8 + 80) + 1024
 
 
 def latent_plan(ctx, num_heads: int, tile_rows: int = LATENT_TILE_ROWS, without=()):
@@ -324,11 +333,13 @@ def paged_latent_attention(q, pages, cache, out, ctx, num_heads: int, wide: int,
         lib = _latent_lib()
         # portions of prompts: tiles of 64 rows (two 16-row tiles per warp, half the key traffic per row) where they fit
         tile_rows = 64 if USE_LATENT_WIDE_TILES and ctx.max_q_len * num_heads >= 64 and lib.mm_attention_latent_tile_rows(wide) == 64 else LATENT_TILE_ROWS
+        if ctx.max_q_len * num_heads <= LATENT_SMALL_TILE_ROWS:      # single tokens of few heads: no rows of padding, two CTAs per SM
+            tile_rows = LATENT_SMALL_TILE_ROWS
         tiles, n_tiles = latent_plan(ctx, num_heads, tile_rows, without)
         keys = min(window, ctx.max_kv_len) if window > 0 else ctx.max_kv_len
-        splits = 1
-        if n_tiles < SINK_TARGET_CTAS // 2:
-            splits = max(1, min(-(-SINK_TARGET_CTAS // n_tiles), -(-keys // (4 * LATENT_KEYS)), SINK_MAX_SPLITS))
+        # as many CTAs as are resident at once (two per SM where two tiles fit its memory): a second wave costs a whole pass
+        resident = 148 * max(1, min(2, (227 << 10) // latent_tile_bytes(wide, tile_rows)))
+        splits = max(1, min(resident // max(1, n_tiles), -(-keys // LATENT_SPLIT_KEYS), LATENT_MAX_SPLITS))
         n_rows = q.shape[0] * num_heads
         part_o = part_ml = None
         if splits > 1:
