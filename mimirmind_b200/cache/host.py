@@ -25,6 +25,7 @@ _PROTOTYPES = {
     "mmh_alloc_check": (I, [P]),
     "mmh_alloc_stat": (L, [P, I]),
     "mmh_cache_create": (P, [I, PI, PI, I, I]),
+    "mmh_cache_set_masks": (I, [P, I, I, PI]),
     "mmh_cache_destroy": (None, [P]),
     "mmh_cache_has": (I, [P, L]),
     "mmh_cache_add": (I, [P, L]),

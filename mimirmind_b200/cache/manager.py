@@ -1,7 +1,7 @@
 """Cache manager: per-request block tables over page pools, and slots for fixed-size state.
 
 Layers whose mixers keep keys and values are sorted into *groups* by what they need (head
-geometry, and whether they look at every earlier token or at a window).  Each group has
+geometry, and which earlier tokens they and the entries that read their cache look at).  Each group has
 its own page pool and each request one block table per group, shared by the group's
 layers.  A request also owns one *state slot*: an index into per-layer arrays of
 fixed-size state (the reference's ``SsmState [layers, nSeq, elems]`` slab, zeroed when a
@@ -12,8 +12,8 @@ count only after ``commit``, src/runtime/KvCache.hpp:90-103):
   ``reserve(request, new_len)``  pages for positions [len, new_len) in every group, all or
                                  nothing (src/runtime/serving/PagedKvSequence.cpp:41-74)
   ... the step writes K/V at [len, new_len) ...
-  ``commit(request, new_len)``   the tokens count; a windowed group gives back the pages
-                                 that no later query can reach
+  ``commit(request, new_len)``   the tokens count; a group whose readers look back over
+                                 a bounded stretch gives back the pages that no later query can reach
   ``release(request)``           everything goes back (src/runtime/serving/PagedKvSequence.cpp:76-87)
 
 Pure host logic, in C++ (``csrc/host/runtime.cpp``); this module is its Python face and maps the caller's request
@@ -47,6 +47,9 @@ class GroupSpec:
     # what an entry keeps per token: (name, shape per token, dtype name or None for the run's dtype); empty means
     # keys and values of (num_kv_heads, head_dim)
     arrays: Tuple[Tuple[str, Tuple[int, ...], Optional[str]], ...] = ()
+    # which earlier tokens the group's readers look at, one (window, chunk, keep) per kind of reader: the last ``window``, the own
+    # run of ``chunk`` tokens (0: no limit), and the first ``keep``; empty means (window, 0, 0)
+    masks: Tuple[Tuple[int, int, int], ...] = ()
 
     def token_arrays(self) -> Tuple[Tuple[str, Tuple[int, ...], Optional[str]], ...]:
         return self.arrays or (("k", (self.num_kv_heads, self.head_dim), None), ("v", (self.num_kv_heads, self.head_dim), None))
@@ -69,6 +72,9 @@ class CacheManager:
                                              page_size, max_requests)
         if not self._h:
             raise CacheError("the cache manager could not be created")
+        for i, g in enumerate(groups):
+            if g.masks and self._lib.mmh_cache_set_masks(self._h, i, len(g.masks), host.int_array([int(x) for m in g.masks for x in m])) != 0:
+                raise CacheError(host.last_error())
         self.max_requests = max_requests
         self.allocators: Dict[str, PageAllocator] = {
             g.name: PageAllocator(0, _borrowed=self._lib.mmh_cache_allocator(self._h, i), _owner=self) for i, g in enumerate(groups)}

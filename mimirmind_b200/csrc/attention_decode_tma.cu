@@ -17,6 +17,10 @@
 // output columns, reading the partials of its peers through distributed shared memory, and writes bf16 output:
 // no scratch in global memory and no merge launch.  Every thread of every CTA reaches both cluster barriers on
 // every path (a CTA without keys, a failed wait), so the barriers cannot be left waiting.
+//
+// The keys a query sees may also be its own run of tokens, and the first tokens of the sequence beside either (KeyMask): the
+// kept tokens' tiles then stand in front of the stretch's in the range that is cut into splits.  A head's output may be
+// multiplied by the logistic of a number per token (`gate`; not in the form that leaves partial results in global memory).
 #include "tcgen05.cuh"
 
 namespace {
@@ -120,8 +124,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
                             const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
                             float* __restrict__ part_ml, const int32_t* __restrict__ items, const int32_t* __restrict__ positions,
                             const int32_t* __restrict__ token_req, const int32_t* __restrict__ block_table, int table_width,
-                            int page_size, int H, int G, int window, float scale_log2, int split_len, int max_splits,
-                            int sink, int* __restrict__ err) {
+                            int page_size, int H, int G, KeyMask mask, float scale_log2, int split_len, int max_splits,
+                            int sink, const float* __restrict__ gate, int gate_ld, int* __restrict__ err) {
     constexpr int KSTEPS = HD / 16;
     constexpr int NT_O = HD / 8;
     constexpr int HALVES = HD / 64;
@@ -136,7 +140,9 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
     const int t = items ? items[item] : item;
     const int pos = positions[t];
     const int hi = pos + 1;
-    const int lo = (window > 0 && hi > window) ? hi - window : 0;
+    const int key_lo0 = mask_low(mask, pos), keep = mask.keep;
+    const TileWalk walk = tile_walk(key_lo0, keep, DT_KT);
+    const int lo = walk.n_kept > 0 ? walk.begin() * DT_KT : key_lo0;     // where the numbered range begins
     const SplitRange sp = split_range(lo, hi, split_len, max_splits);
     const bool has_keys = split >= sp.first && split <= sp.last;
     if (!CLUSTER && !has_keys) return;
@@ -189,8 +195,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
         // latency, between every two tiles
         auto page_of = [&](int kt) -> int {
             if (kt >= kt_end || j >= pages_per_tile) return -1;
-            const int key_lo = kt * DT_KT + j * page_size;
-            return (key_lo < k_end && key_lo + page_size > k_begin) ? table[kt * pages_per_tile + j] : -1;
+            const int kr = walk.real(kt), key_lo = kr * DT_KT + j * page_size;
+            return (key_lo < hi && (key_lo + page_size > key_lo0 || key_lo < keep)) ? table[kr * pages_per_tile + j] : -1;
         };
         constexpr int AHEAD = 4;
         int ahead[AHEAD];
@@ -243,8 +249,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
         const uint32_t ph = (it / STAGES) & 1;
         if (!mbar_wait(smem_u32(&ctl->full[s]), ph, abort_flag)) { ok = false; break; }
         const uint32_t tK = smem_u32(sK + s * TILE), tV = smem_u32(sV + s * TILE);
-        const int key0 = kt * DT_KT + warp * 16;                 // this warp's 16 keys
-        if (key0 < k_end && key0 + 16 > k_begin) {
+        const int key0 = walk.real(kt) * DT_KT + warp * 16;      // this warp's 16 keys
+        if (key0 < hi && (key0 + 16 > key_lo0 || key0 < keep)) {
             float sc[2][4];
             sc[0][0] = sc[0][1] = sc[0][2] = sc[0][3] = 0.0f;
             sc[1][0] = sc[1][1] = sc[1][2] = sc[1][3] = 0.0f;
@@ -262,7 +268,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int key = key0 + j * 8 + (lane & 3) * 2 + (e & 1);
-                    const float v = (key >= k_begin && key < k_end) ? sc[j][e] * scale_log2 : -INFINITY;
+                    const float v = ((key >= key_lo0 || key < keep) && key < hi) ? sc[j][e] * scale_log2 : -INFINITY;
                     sc[j][e] = v;
                     if (e >= 2) mx_hi = fmaxf(mx_hi, v); else mx_lo = fmaxf(mx_lo, v);
                 }
@@ -367,7 +373,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
             }
         } else if (single) {
             if (sink) add_sink(mu, l, acc);
-            out[((size_t)t * H + h) * HD + col] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+            out[((size_t)t * H + h) * HD + col] = __float2bfloat16_rn((l > 0.0f ? acc / l : 0.0f) * head_gate(gate, gate_ld, t, h));
         } else {
             const size_t p = ((size_t)item * H + h) * max_splits + split;
             part_o[p * HD + col] = acc;
@@ -405,7 +411,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
                 }
             }
             if (sink) add_sink(mu, l, acc);
-            out[((size_t)t * H + g * qpg + r) * HD + col] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+            out[((size_t)t * H + g * qpg + r) * HD + col] =
+                __float2bfloat16_rn((l > 0.0f ? acc / l : 0.0f) * head_gate(gate, gate_ld, t, g * qpg + r));
         }
         cluster_sync_all();                            // peers may still be reading this CTA's shared memory
     }
@@ -414,8 +421,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
 template <int HD, int STAGES, bool CLUSTER>
 int launch_decode_tma(const CUtensorMap& tk, const CUtensorMap& tv, const void* q, void* out, void* part_o, void* part_ml,
                       const void* items, int n_items, const void* positions, const void* token_req, const void* table,
-                      int table_width, int page_size, int H, int G, int window, float scale, int split_len, int max_splits,
-                      int sink, int* err, cudaStream_t s) {
+                      int table_width, int page_size, int H, int G, KeyMask mask, float scale, int split_len, int max_splits,
+                      int sink, const void* gate, int gate_ld, int* err, cudaStream_t s) {
     constexpr int TILE = DT_KT * HD * 2;
     const size_t smem = (size_t)2 * STAGES * TILE + sizeof(DecCtl<STAGES>);
     static bool configured = false;
@@ -440,8 +447,8 @@ int launch_decode_tma(const CUtensorMap& tk, const CUtensorMap& tv, const void* 
     cfg.numAttrs = CLUSTER ? 1 : 0;
     cudaLaunchKernelEx(&cfg, attention_decode_tma_kernel<HD, STAGES, CLUSTER>, tk, tv, (const __nv_bfloat16*)q, (__nv_bfloat16*)out,
                        (float*)part_o, (float*)part_ml, (const int32_t*)items, (const int32_t*)positions, (const int32_t*)token_req,
-                       (const int32_t*)table, table_width, page_size, H, G, window, scale * 1.4426950408889634f, split_len,
-                       max_splits, sink, err);
+                       (const int32_t*)table, table_width, page_size, H, G, mask, scale * 1.4426950408889634f, split_len,
+                       max_splits, sink, (const float*)gate, gate_ld, err);
     MM_CHECK_LAUNCH();
     return MM_OK;
 }
@@ -483,8 +490,8 @@ int max_active_clusters(int cluster_size, int* out) {
 static int attention_decode_tma_launch(const void* q, const void* k_pages, const void* v_pages, void* out, void* part_o,
                                        void* part_ml, const void* items, int n_items, const void* positions,
                                        const void* token_req, const void* block_table, int table_width, int page_size,
-                                       int num_pages, int H, int G, int hd, int window, float scale, int split_len,
-                                       int max_splits, int stages, int cluster, int sink, void* err, void* stream) {
+                                       int num_pages, int H, int G, int hd, KeyMask mask, float scale, int split_len,
+                                       int max_splits, int stages, int cluster, int sink, const void* gate, int gate_ld, void* err, void* stream) {
     MM_REQUIRE(hd == 64 || hd == 128, "attention_decode_tma: built for head_dim 64 and 128");
     MM_REQUIRE(n_items >= 0 && H > 0 && G > 0 && H % G == 0 && H / G <= 16 && num_pages > 0, "attention_decode_tma: bad head counts");
     MM_REQUIRE(page_size >= 8 && page_size <= 64 && (64 % page_size) == 0, "attention_decode_tma: page_size must be 8, 16, 32 or 64");
@@ -492,6 +499,8 @@ static int attention_decode_tma_launch(const void* q, const void* k_pages, const
     MM_REQUIRE(cluster || max_splits == 1 || (part_o != nullptr && part_ml != nullptr), "attention_decode_tma: scratch missing");
     MM_REQUIRE(!cluster || (max_splits >= 2 && max_splits <= 8), "attention_decode_tma: a cluster merges 2 to 8 splits");
     MM_REQUIRE(stages == 3 || stages == 6, "attention_decode_tma: stages must be 3 or 6");
+    MM_REQUIRE(mask.window >= 0 && mask.chunk >= 0 && mask.keep >= 0 && (gate == nullptr || gate_ld >= H), "attention_decode_tma: bad mask or gate");
+    MM_REQUIRE(split_len == 0 || (mask.chunk == 0 && mask.keep == 0), "attention_decode_tma: splits of a fixed length take a plain window");
     if (n_items == 0) return MM_OK;
     CUtensorMap tk, tv;
     const long long pool_rows = (long long)num_pages * G * page_size;
@@ -501,7 +510,7 @@ static int attention_decode_tma_launch(const void* q, const void* k_pages, const
     }
     cudaStream_t s = (cudaStream_t)stream;
 #define MM_DT(HDV, ST, CL) launch_decode_tma<HDV, ST, CL>(tk, tv, q, out, part_o, part_ml, items, n_items, positions, token_req, block_table, \
-                                                          table_width, page_size, H, G, window, scale, split_len, max_splits, sink, (int*)err, s)
+                                                          table_width, page_size, H, G, mask, scale, split_len, max_splits, sink, gate, gate_ld, (int*)err, s)
     if (cluster) return hd == 128 ? MM_DT(128, 3, true) : MM_DT(64, 3, true);
     if (hd == 128) return stages == 3 ? MM_DT(128, 3, false) : MM_DT(128, 6, false);
     return stages == 3 ? MM_DT(64, 3, false) : MM_DT(64, 6, false);
@@ -514,20 +523,22 @@ MM_EXPORT int mm_attention_decode_tma_bf16(const void* q, const void* k_pages, c
                                            int num_pages, int H, int G, int hd, int window, float scale, int split_len,
                                            int max_splits, int stages, int cluster, void* err, void* stream) {
     return attention_decode_tma_launch(q, k_pages, v_pages, out, part_o, part_ml, items, n_items, positions, token_req, block_table,
-                                       table_width, page_size, num_pages, H, G, hd, window, scale, split_len, max_splits, stages,
-                                       cluster, 0, err, stream);
+                                       table_width, page_size, num_pages, H, G, hd, KeyMask{window, 0, 0}, scale, split_len, max_splits, stages,
+                                       cluster, 0, nullptr, 0, err, stream);
 }
 
-// The same with a softmax sink (one added to every row's denominator), for the two forms that finish a row inside the
+// The same with a softmax sink (one added to every row's denominator), any mask and a gate per head (fp32 [n_tokens, gate_ld] or
+// null), for the two forms that finish a row inside the
 // kernel: one split per token, or the splits of a token as one cluster.
 MM_EXPORT int mm_attention_decode_tma_bf16_sink(const void* q, const void* k_pages, const void* v_pages, void* out, const void* items,
                                                 int n_items, const void* positions, const void* token_req, const void* block_table,
                                                 int table_width, int page_size, int num_pages, int H, int G, int hd, int window,
-                                                float scale, int max_splits, int cluster, int sink, void* err, void* stream) {
+                                                int chunk, int keep, float scale, int max_splits, int cluster, int sink, const void* gate, int gate_ld,
+                                                void* err, void* stream) {
     MM_REQUIRE(cluster || max_splits == 1, "attention_decode_tma: with a sink the splits of a token are one cluster");
     return attention_decode_tma_launch(q, k_pages, v_pages, out, nullptr, nullptr, items, n_items, positions, token_req, block_table,
-                                       table_width, page_size, num_pages, H, G, hd, window, scale, 0, max_splits, 3, cluster, sink, err,
-                                       stream);
+                                       table_width, page_size, num_pages, H, G, hd, KeyMask{window, chunk, keep}, scale, 0, max_splits, 3, cluster,
+                                       sink, gate, gate_ld, err, stream);
 }
 
 // Clusters of `cluster_size` (2..8) CTAs of the cluster variant that fit on the current device at the same time; a

@@ -1,7 +1,8 @@
 // Windowed attention with a softmax sink, and keys and values of different sizes.
 //
 //   q [n, H, dk], keys [.., G, dk], values [.., G, dv]; query head h reads kv head h / (H / G);
-//   a query at absolute position a sees keys max(0, a + 1 - W) .. a (W = 0: all);
+//   a query at absolute position a sees keys max(0, a + 1 - W) .. a (W = 0: all), or what another KeyMask lets it see
+//   (own runs of tokens, kept first tokens); a head's output may be multiplied by the logistic of a number per token;
 //   s_j = (q . k_j) * scale;  p_j = exp(s_j) / (sink + sum_i exp(s_i)),  sink = 1 or 0;  o = sum_j p_j v_j.
 //
 // The sink is a key of score 0 that has no value: it only takes its share of the weights.  The fp32-arithmetic
@@ -185,9 +186,9 @@ __global__ void attention_sink_generic_kernel(const T* __restrict__ q, const T* 
                                               const T* __restrict__ v_pages, TO* __restrict__ out,
                                               const int32_t* __restrict__ positions, const int32_t* __restrict__ token_req,
                                               const int32_t* __restrict__ block_table, int table_width, int page_size,
-                                              int n_tokens, int H, int G, int dk, int dv, int window, float scale, int sink,
+                                              int n_tokens, int H, int G, int dk, int dv, KeyMask mask, float scale, int sink,
                                               const float* __restrict__ sink_logit, const float* __restrict__ dist_bias, int dist_max,
-                                              float softcap, int Gv, int v_row) {
+                                              float softcap, int Gv, int v_row, const float* __restrict__ gate, int gate_ld) {
     extern __shared__ float q_smem[];  // [warps][dk]
     const int warps_per_block = blockDim.x >> 5;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -198,7 +199,7 @@ __global__ void attention_sink_generic_kernel(const T* __restrict__ q, const T* 
     const int pos = positions[t];
     const int32_t* table = block_table + (size_t)token_req[t] * table_width;
     const int hi = pos + 1;
-    const int lo = (window > 0 && hi > window) ? hi - window : 0;
+    const int lo = mask_low(mask, pos);
 
     float* qs = q_smem + warp * dk;
     const T* qrow = q + ((size_t)t * H + h) * dk;
@@ -216,9 +217,11 @@ __global__ void attention_sink_generic_kernel(const T* __restrict__ q, const T* 
     const size_t v_head = (size_t)(g % Gv) * page_size * v_row, v_stride = (size_t)Gv * page_size * v_row;
     const float inv_cap = softcap > 0.0f ? 1.0f / softcap : 0.0f;
 
-    for (int c = (lo / 32) * 32; c < hi; c += 32) {
+    const TileWalk walk = tile_walk(lo, mask.keep, 32);
+    for (int ct = walk.begin(); ct * 32 < hi; ++ct) {
+        const int c = walk.real(ct) * 32;
         const int j = c + lane;
-        const bool valid = (j >= lo) && (j < hi);
+        const bool valid = (j >= lo || j < mask.keep) && (j < hi);
         float s = -INFINITY;
         if (valid) {
             const int page = table[j / page_size];
@@ -237,7 +240,7 @@ __global__ void attention_sink_generic_kernel(const T* __restrict__ q, const T* 
         for (int a = 0; a < SINK_MAX_ACC; ++a) acc[a] *= alpha;
         for (int jj = 0; jj < 32; ++jj) {
             const int key = c + jj;
-            if (key < lo || key >= hi) continue;  // uniform over the warp
+            if ((key < lo && key >= mask.keep) || key >= hi) continue;  // uniform over the warp
             const float pj = __shfl_sync(0xffffffffu, p, jj);
             const int page = table[key / page_size];
             const T* vr = v_pages + (size_t)page * v_stride + v_head + (size_t)(key % page_size) * v_row;
@@ -249,7 +252,7 @@ __global__ void attention_sink_generic_kernel(const T* __restrict__ q, const T* 
         }
         m = m_new;
     }
-    const float inv_l = (l > 0.0f) ? 1.0f / l : 0.0f;
+    const float inv_l = ((l > 0.0f) ? 1.0f / l : 0.0f) * head_gate(gate, gate_ld, t, h);
     TO* orow = out + ((size_t)t * H + h) * dv;
 #pragma unroll
     for (int a = 0; a < SINK_MAX_ACC; ++a) {
@@ -260,14 +263,16 @@ __global__ void attention_sink_generic_kernel(const T* __restrict__ q, const T* 
 
 MM_EXPORT int mm_attention_sink_generic(const void* q, const void* k_pages, const void* v_pages, void* out, int dtype,
                                         const void* positions, const void* token_req, const void* block_table,
-                                        int table_width, int page_size, int n_tokens, int H, int G, int dk, int dv, int window,
-                                        float scale, int sink, const void* sink_logit, const void* dist_bias, int dist_max, float softcap,
-                                        int Gv, int v_row, int out_f32, void* stream) {
+                                        int table_width, int page_size, int n_tokens, int H, int G, int dk, int dv, int window, int chunk,
+                                        int keep, float scale, int sink, const void* sink_logit, const void* dist_bias, int dist_max, float softcap,
+                                        int Gv, int v_row, const void* gate, int gate_ld, int out_f32, void* stream) {
     MM_REQUIRE(dist_bias == nullptr || dist_max >= 0, "attention: the distance table needs at least one row");
     MM_REQUIRE(Gv >= 1 && G % Gv == 0 && v_row >= dv && softcap >= 0.0f, "attention: value heads must divide the key heads, a value row holds at least dv numbers");
     MM_REQUIRE(n_tokens >= 0 && H > 0 && G > 0 && dk > 0 && dv > 0 && H % G == 0, "attention: heads must be a positive multiple of kv heads");
     MM_REQUIRE(dv <= 32 * SINK_MAX_ACC && dk <= 2048, "attention: value size above 512 or key size above 2048 is not supported");
-    MM_REQUIRE(page_size > 0 && table_width > 0 && window >= 0, "attention: bad page geometry or window");
+    MM_REQUIRE(page_size > 0 && table_width > 0 && window >= 0 && chunk >= 0 && keep >= 0, "attention: bad page geometry or mask");
+    MM_REQUIRE(gate == nullptr || gate_ld >= H, "attention: one gate per head");
+    const KeyMask mask = {window, chunk, keep};
     if (n_tokens == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
     const int warps = 4;
@@ -277,18 +282,18 @@ MM_EXPORT int mm_attention_sink_generic(const void* q, const void* k_pages, cons
     if (dtype == MM_F32)
         mm_launch(attention_sink_generic_kernel<float>, dim3(blocks), dim3(warps * 32), smem, s, (const float*)q, (const float*)k_pages,
                   (const float*)v_pages, (float*)out, (const int32_t*)positions, (const int32_t*)token_req,
-                  (const int32_t*)block_table, table_width, page_size, n_tokens, H, G, dk, dv, window, scale, sink,
-                  (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, v_row);
+                  (const int32_t*)block_table, table_width, page_size, n_tokens, H, G, dk, dv, mask, scale, sink,
+                  (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, v_row, (const float*)gate, gate_ld);
     else if (dtype == MM_BF16 && out_f32)      // the result is not rounded: what follows takes a difference of heads
         mm_launch(attention_sink_generic_kernel<__nv_bfloat16, float>, dim3(blocks), dim3(warps * 32), smem, s, (const __nv_bfloat16*)q,
                   (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, (float*)out, (const int32_t*)positions,
-                  (const int32_t*)token_req, (const int32_t*)block_table, table_width, page_size, n_tokens, H, G, dk, dv, window,
-                  scale, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, v_row);
+                  (const int32_t*)token_req, (const int32_t*)block_table, table_width, page_size, n_tokens, H, G, dk, dv, mask,
+                  scale, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, v_row, (const float*)gate, gate_ld);
     else if (dtype == MM_BF16)
         mm_launch(attention_sink_generic_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, s, (const __nv_bfloat16*)q,
                   (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, (__nv_bfloat16*)out, (const int32_t*)positions,
-                  (const int32_t*)token_req, (const int32_t*)block_table, table_width, page_size, n_tokens, H, G, dk, dv, window,
-                  scale, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, v_row);
+                  (const int32_t*)token_req, (const int32_t*)block_table, table_width, page_size, n_tokens, H, G, dk, dv, mask,
+                  scale, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, v_row, (const float*)gate, gate_ld);
     else
         MM_REQUIRE(false, "attention: dtype must be float32 or bfloat16");
     MM_CHECK_LAUNCH();

@@ -3,6 +3,10 @@
 //
 //   s_j = (q . k_j) * scale;  p_j = exp(s_j) / (sink + sum_i exp(s_i));  o = sum_j p_j v_j
 //
+// The keys a query sees may also be its own run of tokens, and the first tokens of the sequence beside either (KeyMask): the
+// walk over key tiles then starts with the kept tokens' tiles.  A head's output may be multiplied by the logistic of a number
+// per token (`gate`).
+//
 // The sink is a key of score 0 without a value: the running softmax starts from (maximum 0, mass 1, nothing
 // accumulated) instead of (-inf, 0, 0).
 //
@@ -23,14 +27,15 @@
 #define SATT_THREADS 128  // 4 warps
 #define SDEC_STAGES 3
 
-// 64 key rows [64][DK + 8] and the same 64 value rows [64][DV + 8] of one KV head; rows outside [lo, hi) are zero.
+// 64 key rows [64][DK + 8] and the same 64 value rows [64][DV + 8] of one KV head; rows outside
+// [lo, hi) and not among the first `keep` keys are zero.
 // Warp w fetches rows 16 w .. 16 w + 15: its first sixteen lanes look up one row's page and place each, and every lane
 // takes those from the row's lane for the 16-byte pieces it copies (one table read per row, not per piece).  Every
 // thread of the CTA must call this together.
 template <int DK, int DV>
 __device__ __forceinline__ void load_kv_tile2(__nv_bfloat16* dK, __nv_bfloat16* dV, const __nv_bfloat16* __restrict__ kpool,
                                               const __nv_bfloat16* __restrict__ vpool, const int32_t* __restrict__ table,
-                                              int key0, int lo, int hi, int G, int g, int page_size, int page_shift, int Gv) {
+                                              int key0, int lo, int hi, int keep, int G, int g, int page_size, int page_shift, int Gv) {
     constexpr int KS = DK + 8, VS = DV + 8, KC = DK / 8, VC = DV / 8;
     static_assert(SATT_THREADS == 128 && SKT == 64 && (16 * KC) % 32 == 0 && (16 * VC) % 32 == 0, "a warp per 16 rows");
     const int gv = g % Gv;      // the value pool has Gv heads; key head g reads value head g mod Gv
@@ -38,7 +43,7 @@ __device__ __forceinline__ void load_kv_tile2(__nv_bfloat16* dK, __nv_bfloat16* 
     int page = -1, slot = 0;
     {
         const int key = key0 + warp * 16 + (lane & 15);
-        if (key >= lo && key < hi) {
+        if ((key >= lo || key < keep) && key < hi) {
             const int pidx = page_shift >= 0 ? (key >> page_shift) : (key / page_size);
             slot = key - pidx * page_size;
             page = table[pidx];
@@ -73,8 +78,9 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
     const __nv_bfloat16* __restrict__ v_pages, __nv_bfloat16* __restrict__ out, float* __restrict__ out32,
     const int32_t* __restrict__ tiles,
-    const int32_t* __restrict__ block_table, int table_width, int page_size, int H, int G, int window, float scale_log2,
-    int sink, const float* __restrict__ sink_logit, const float* __restrict__ dist_bias, int dist_max, float softcap, int Gv) {
+    const int32_t* __restrict__ block_table, int table_width, int page_size, int H, int G, KeyMask mask, float scale_log2,
+    int sink, const float* __restrict__ sink_logit, const float* __restrict__ dist_bias, int dist_max, float softcap, int Gv,
+    const float* __restrict__ gate, int gate_ld) {
     constexpr int KS = DK + 8, VS = DV + 8;
     constexpr int KSTEPS = DK / 16;
     constexpr int NT_O = DV / 8;
@@ -91,8 +97,9 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
     const int hi_all = pos0 + n_rows;                                     // exclusive
-    const int lo_all = (window > 0 && pos0 + 1 > window) ? pos0 + 1 - window : 0;
-    const int kt_begin = lo_all / SKT, kt_end = (hi_all + SKT - 1) / SKT;
+    const int lo_all = mask_low(mask, pos0), keep = mask.keep;
+    const TileWalk walk = tile_walk(lo_all, keep, SKT);
+    const int kt_begin = walk.begin(), kt_end = (hi_all + SKT - 1) / SKT;
 
     for (int c = threadIdx.x; c < 64 * (DK / 8); c += SATT_THREADS) {
         const int r = c / (DK / 8), part = c - r * (DK / 8);
@@ -101,7 +108,7 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
         *reinterpret_cast<uint4*>(sQ + r * KS + part * 8) = v;
     }
     const int page_shift = (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;
-    load_kv_tile2<DK, DV>(sK, sV, k_pages, v_pages, table, kt_begin * SKT, lo_all, hi_all, G, g, page_size, page_shift, Gv);
+    load_kv_tile2<DK, DV>(sK, sV, k_pages, v_pages, table, walk.real(kt_begin) * SKT, lo_all, hi_all, keep, G, g, page_size, page_shift, Gv);
     cp_async_commit();
     __syncthreads();
 
@@ -115,8 +122,8 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
     }
     const int r_lo = warp * 16 + (lane >> 2), r_hi = r_lo + 8;
     const int pos_lo = pos0 + r_lo, pos_hi = pos0 + r_hi;
-    const int wlo_lo = (window > 0 && pos_lo + 1 > window) ? pos_lo + 1 - window : 0;
-    const int wlo_hi = (window > 0 && pos_hi + 1 > window) ? pos_hi + 1 - window : 0;
+    const int wlo_lo = mask_low(mask, pos_lo), wlo_hi = mask_low(mask, pos_hi);
+    const int wlo_first = mask_low(mask, pos0 + warp * 16), wlo_last = mask_low(mask, pos0 + warp * 16 + 15);
     const bool valid_lo = r_lo < n_rows, valid_hi = r_hi < n_rows;
 
     float o[NT_O][4];
@@ -136,8 +143,8 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
     for (int kt = kt_begin; kt < kt_end; ++kt) {
         const int buf = (kt - kt_begin) & 1;
         if (kt + 1 < kt_end) {
-            load_kv_tile2<DK, DV>(sK + (buf ^ 1) * SKT * KS, sV + (buf ^ 1) * SKT * VS, k_pages, v_pages, table, (kt + 1) * SKT,
-                                  lo_all, hi_all, G, g, page_size, page_shift, Gv);
+            load_kv_tile2<DK, DV>(sK + (buf ^ 1) * SKT * KS, sV + (buf ^ 1) * SKT * VS, k_pages, v_pages, table, walk.real(kt + 1) * SKT,
+                                  lo_all, hi_all, keep, G, g, page_size, page_shift, Gv);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -146,10 +153,10 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
         __syncthreads();
         const __nv_bfloat16* tK = sK + buf * SKT * KS;
         const __nv_bfloat16* tV = sV + buf * SKT * VS;
-        const int key0 = kt * SKT;
+        const int key0 = walk.real(kt) * SKT;
         // a warp whose rows all lie before this tile, or whose windows all begin after it, has nothing to do in it
         const bool warp_active = (pos0 + warp * 16 + 15 >= key0) && (warp * 16 < n_rows) &&
-                                 (window == 0 || key0 + SKT - 1 >= pos0 + warp * 16 + 1 - window);
+                                 (key0 + SKT - 1 >= wlo_first || key0 < keep);
         if (warp_active) {
             float s[8][4];
 #pragma unroll
@@ -167,7 +174,7 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
                 }
             }
             const bool interior = (key0 + SKT - 1 <= pos0 + warp * 16) && (warp * 16 + 15 < n_rows) &&
-                                  (window == 0 || key0 >= pos0 + warp * 16 + 16 - window);
+                                  key0 >= wlo_last;
             float mx_lo = m_lo, mx_hi = m_hi;
             if (ext) {
                 // every key of the tile at least dist_max behind every row of the warp: one bias for all
@@ -194,7 +201,7 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
                     for (int e = 0; e < 4; ++e) {
                         const int key = key0 + j * 8 + (lane & 3) * 2 + (e & 1);
                         const bool hi_row = e >= 2;
-                        const bool ok = hi_row ? (valid_hi && key <= pos_hi && key >= wlo_hi) : (valid_lo && key <= pos_lo && key >= wlo_lo);
+                        const bool ok = hi_row ? (valid_hi && key <= pos_hi && (key >= wlo_hi || key < keep)) : (valid_lo && key <= pos_lo && (key >= wlo_lo || key < keep));
                         if (!ok) s[j][e] = -INFINITY;
                     }
                 }
@@ -249,7 +256,11 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_prefill_kernel(
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
-    const float inv_lo = l_lo > 0.0f ? 1.0f / l_lo : 0.0f, inv_hi = l_hi > 0.0f ? 1.0f / l_hi : 0.0f;
+    float inv_lo = l_lo > 0.0f ? 1.0f / l_lo : 0.0f, inv_hi = l_hi > 0.0f ? 1.0f / l_hi : 0.0f;
+    if (gate != nullptr) {
+        if (valid_lo) inv_lo *= head_gate(gate, gate_ld, row0 + r_lo, h);
+        if (valid_hi) inv_hi *= head_gate(gate, gate_ld, row0 + r_hi, h);
+    }
 #pragma unroll
     for (int j = 0; j < NT_O; ++j) {
         const int col = j * 8 + (lane & 3) * 2;
@@ -273,8 +284,8 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
     const __nv_bfloat16* __restrict__ v_pages, __nv_bfloat16* __restrict__ out, float* __restrict__ out32, float* __restrict__ part_o,
     float* __restrict__ part_ml, const int32_t* __restrict__ items,
     const int32_t* __restrict__ positions, const int32_t* __restrict__ token_req, const int32_t* __restrict__ block_table,
-    int table_width, int page_size, int H, int G, int window, float scale_log2, int sink, const float* __restrict__ sink_logit,
-    const float* __restrict__ dist_bias, int dist_max, float softcap, int Gv) {
+    int table_width, int page_size, int H, int G, KeyMask mask, float scale_log2, int sink, const float* __restrict__ sink_logit,
+    const float* __restrict__ dist_bias, int dist_max, float softcap, int Gv, const float* __restrict__ gate, int gate_ld) {
     constexpr int KS = DK + 8, VS = DV + 8;
     constexpr int KSTEPS = DK / 16;
     constexpr int NT_O = DV / 8;
@@ -287,10 +298,11 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
     const int t = items ? items[item] : item;
     const int pos = positions[t];
     const int k_end = pos + 1;
-    const int k_begin = (window > 0 && k_end > window) ? k_end - window : 0;
+    const int k_begin = mask_low(mask, pos), keep = mask.keep;
+    const TileWalk walk = tile_walk(k_begin, keep, SKT);
     // gridDim.z CTAs share the token's key tiles evenly (a CTA may get none: it posts an empty partial result)
     const int n_splits = gridDim.z, split = blockIdx.z;
-    const int kt_first = k_begin / SKT, kt_last = (k_end + SKT - 1) / SKT;
+    const int kt_first = walk.begin(), kt_last = (k_end + SKT - 1) / SKT;
     const int per_split = (kt_last - kt_first + n_splits - 1) / n_splits;
     const int kt_begin = min(kt_last, kt_first + split * per_split), kt_end = min(kt_last, kt_begin + per_split);
     const int32_t* table = block_table + (size_t)token_req[t] * table_width;
@@ -301,8 +313,8 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
 #pragma unroll
     for (int st = 0; st < SDEC_STAGES - 1; ++st) {
         if (kt_begin + st < kt_end)
-            load_kv_tile2<DK, DV>(sK + st * SKT * KS, sV + st * SKT * VS, k_pages, v_pages, table, (kt_begin + st) * SKT, k_begin, k_end,
-                                  G, g, page_size, page_shift, Gv);
+            load_kv_tile2<DK, DV>(sK + st * SKT * KS, sV + st * SKT * VS, k_pages, v_pages, table, walk.real(kt_begin + st) * SKT, k_begin, k_end,
+                                  keep, G, g, page_size, page_shift, Gv);
         cp_async_commit();
     }
     uint32_t qf[KSTEPS][4];
@@ -330,7 +342,7 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
             const int nxt = kt + SDEC_STAGES - 1;
             if (nxt < kt_end) {
                 const int nb = (nxt - kt_begin) % SDEC_STAGES;
-                load_kv_tile2<DK, DV>(sK + nb * SKT * KS, sV + nb * SKT * VS, k_pages, v_pages, table, nxt * SKT, k_begin, k_end, G, g,
+                load_kv_tile2<DK, DV>(sK + nb * SKT * KS, sV + nb * SKT * VS, k_pages, v_pages, table, walk.real(nxt) * SKT, k_begin, k_end, keep, G, g,
                                       page_size, page_shift, Gv);
             }
             cp_async_commit();
@@ -339,8 +351,8 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
         __syncthreads();
         const __nv_bfloat16* tK = sK + buf * SKT * KS + warp * 16 * KS;   // this warp's 16 keys
         const __nv_bfloat16* tV = sV + buf * SKT * VS + warp * 16 * VS;
-        const int key0 = kt * SKT + warp * 16;
-        if (key0 < k_end && key0 + 16 > k_begin) {
+        const int key0 = walk.real(kt) * SKT + warp * 16;
+        if (key0 < k_end && (key0 + 16 > k_begin || key0 < keep)) {
             float s[2][4];
             s[0][0] = s[0][1] = s[0][2] = s[0][3] = 0.0f;
             s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.0f;
@@ -359,7 +371,7 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
                 for (int e = 0; e < 4; ++e) {
                     const int key = key0 + j * 8 + (lane & 3) * 2 + (e & 1);
                     float v = -INFINITY;
-                    if (key >= k_begin && key < k_end) {
+                    if ((key >= k_begin || key < keep) && key < k_end) {
                         // rows of the tile are the query heads of this kv head; the rows beyond them hold zero queries and
                         // scores, whose capped form is zero as well
                         const bool real_row = (lane >> 2) + (e >= 2 ? 8 : 0) < qpg;
@@ -453,7 +465,7 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
         }
         const int h = g * qpg + r;
         if (single) {
-            const float res = l > 0.0f ? acc / l : 0.0f;
+            const float res = (l > 0.0f ? acc / l : 0.0f) * head_gate(gate, gate_ld, t, h);
             if (out32 != nullptr) out32[((size_t)t * H + h) * DV + col] = res;
             else out[((size_t)t * H + h) * DV + col] = __float2bfloat16_rn(res);
         } else {
@@ -470,7 +482,8 @@ __global__ void __launch_bounds__(SATT_THREADS) attention_sink_decode_kernel(
 // The splits of every (item, head) put together in split order, with the sink's share: one block per (item, head).
 __global__ void attention_sink_merge_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ out32, const float* __restrict__ part_o,
                                             const float* __restrict__ part_ml, const int32_t* __restrict__ items, int H, int dv,
-                                            int n_splits, int sink, const float* __restrict__ sink_logit) {
+                                            int n_splits, int sink, const float* __restrict__ sink_logit, const float* __restrict__ gate,
+                                            int gate_ld) {
     const int item = blockIdx.x, h = blockIdx.y;
     const int t = items ? items[item] : item;
     const size_t p0 = ((size_t)item * H + h) * n_splits;
@@ -481,7 +494,7 @@ __global__ void attention_sink_merge_kernel(__nv_bfloat16* __restrict__ out, flo
     const float mu = (m == -INFINITY) ? 0.0f : m;
     float l = with_sink ? exp2f(sink_m - mu) : 0.0f;
     for (int s = 0; s < n_splits; ++s) l += part_ml[(p0 + s) * 2 + 1] * exp2f(part_ml[(p0 + s) * 2] - mu);
-    const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * head_gate(gate, gate_ld, t, h);
     for (int col = threadIdx.x; col < dv; col += blockDim.x) {
         float acc = 0.0f;
         for (int s = 0; s < n_splits; ++s) acc += part_o[(p0 + s) * dv + col] * exp2f(part_ml[(p0 + s) * 2] - mu);
@@ -494,9 +507,9 @@ static const float SINK_LOG2E = 1.4426950408889634f;
 
 template <int DK, int DV>
 static int launch_sink_prefill(const void* q, const void* k, const void* v, void* out, const void* tiles, int n_tiles,
-                               const void* table, int table_width, int page_size, int H, int G, int window, float scale, int sink,
-                               const void* sink_logit, const void* dist_bias, int dist_max, float softcap, int Gv, int out_f32,
-                               cudaStream_t s) {
+                               const void* table, int table_width, int page_size, int H, int G, KeyMask mask, float scale, int sink,
+                               const void* sink_logit, const void* dist_bias, int dist_max, float softcap, int Gv, const void* gate, int gate_ld,
+                               int out_f32, cudaStream_t s) {
     const size_t smem = (size_t)(3 * 64 * (DK + 8) + 2 * 64 * (DV + 8)) * sizeof(__nv_bfloat16);
     auto kernel = attention_sink_prefill_kernel<DK, DV>;
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
@@ -507,7 +520,7 @@ static int launch_sink_prefill(const void* q, const void* k, const void* v, void
     mm_launch(kernel, dim3(H, n_tiles), dim3(SATT_THREADS), smem, s, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k,
               (const __nv_bfloat16*)v, out_f32 ? nullptr : (__nv_bfloat16*)out, out_f32 ? (float*)out : nullptr, (const int32_t*)tiles,
               (const int32_t*)table, table_width, page_size, H, G,
-              window, scale * SINK_LOG2E, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv);
+              mask, scale * SINK_LOG2E, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, (const float*)gate, gate_ld);
     MM_CHECK_LAUNCH();
     return MM_OK;
 }
@@ -516,8 +529,8 @@ template <int DK, int DV>
 static int launch_sink_decode(const void* q, const void* k, const void* v, void* out, void* part_o, void* part_ml, int n_splits,
                               const void* items, int n_items,
                               const void* positions, const void* token_req, const void* table, int table_width, int page_size,
-                              int H, int G, int window, float scale, int sink, const void* sink_logit, const void* dist_bias, int dist_max,
-                              float softcap, int Gv, int out_f32, cudaStream_t s) {
+                              int H, int G, KeyMask mask, float scale, int sink, const void* sink_logit, const void* dist_bias, int dist_max,
+                              float softcap, int Gv, const void* gate, int gate_ld, int out_f32, cudaStream_t s) {
     const size_t kv = (size_t)SDEC_STAGES * 64 * (DK + 8 + DV + 8) * sizeof(__nv_bfloat16);
     const size_t merge = (size_t)(4 * 16 * DV + 4 * 16 * 2) * sizeof(float);
     const size_t smem = kv > merge ? kv : merge;
@@ -530,13 +543,14 @@ static int launch_sink_decode(const void* q, const void* k, const void* v, void*
     mm_launch(kernel, dim3(n_items, G, n_splits), dim3(SATT_THREADS), smem, s, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k,
               (const __nv_bfloat16*)v, out_f32 ? nullptr : (__nv_bfloat16*)out, out_f32 ? (float*)out : nullptr, (float*)part_o,
               (float*)part_ml, (const int32_t*)items,
-              (const int32_t*)positions, (const int32_t*)token_req, (const int32_t*)table, table_width, page_size, H, G, window,
-              scale * SINK_LOG2E, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv);
+              (const int32_t*)positions, (const int32_t*)token_req, (const int32_t*)table, table_width, page_size, H, G, mask,
+              scale * SINK_LOG2E, sink, (const float*)sink_logit, (const float*)dist_bias, dist_max, softcap, Gv, (const float*)gate, gate_ld);
     MM_CHECK_LAUNCH();
     if (n_splits > 1) {
         mm_launch(attention_sink_merge_kernel, dim3(n_items, H), dim3(DV >= 64 ? 64 : 32), 0, s, out_f32 ? nullptr : (__nv_bfloat16*)out,
                   out_f32 ? (float*)out : nullptr, (const float*)part_o,
-                  (const float*)part_ml, (const int32_t*)items, H, DV, n_splits, sink, (const float*)sink_logit);
+                  (const float*)part_ml, (const int32_t*)items, H, DV, n_splits, sink, (const float*)sink_logit,
+                  (const float*)gate, gate_ld);
         MM_CHECK_LAUNCH();
     }
     return MM_OK;
@@ -570,15 +584,18 @@ MM_EXPORT int mm_attention_sink_supported(int dk, int dv) {
 
 MM_EXPORT int mm_attention_sink_prefill_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, const void* tiles,
                                              int n_tiles, const void* block_table, int table_width, int page_size, int H, int G,
-                                             int dk, int dv, int window, float scale, int sink, const void* sink_logit, const void* dist_bias,
-                                             int dist_max, float softcap, int Gv, int out_f32, void* stream) {
+                                             int dk, int dv, int window, int chunk, int keep, float scale, int sink, const void* sink_logit,
+                                             const void* dist_bias, int dist_max, float softcap, int Gv, const void* gate, int gate_ld, int out_f32,
+                                             void* stream) {
     MM_REQUIRE(Gv >= 1 && G % Gv == 0 && softcap >= 0.0f, "sink attention: the value heads must divide the key heads");
     MM_REQUIRE(n_tiles >= 0 && H > 0 && G > 0 && H % G == 0, "sink attention: heads must be a positive multiple of kv heads");
-    MM_REQUIRE(page_size > 0 && table_width > 0 && window >= 0 && scale > 0.0f, "sink attention: bad page geometry, window or scale");
+    MM_REQUIRE(page_size > 0 && table_width > 0 && window >= 0 && chunk >= 0 && keep >= 0 && scale > 0.0f, "sink attention: bad page geometry, mask or scale");
+    MM_REQUIRE(gate == nullptr || gate_ld >= H, "sink attention: one gate per head");
+    const KeyMask mask = {window, chunk, keep};
     if (n_tiles == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
-    SINK_DISPATCH(launch_sink_prefill, q, k_pages, v_pages, out, tiles, n_tiles, block_table, table_width, page_size, H, G, window, scale,
-                  sink, sink_logit, dist_bias, dist_max, softcap, Gv, out_f32, s);
+    SINK_DISPATCH(launch_sink_prefill, q, k_pages, v_pages, out, tiles, n_tiles, block_table, table_width, page_size, H, G, mask, scale,
+                  sink, sink_logit, dist_bias, dist_max, softcap, Gv, gate, gate_ld, out_f32, s);
     mm_set_last_error("sink attention: key and value sizes must each be one of 32, 64, 96, 128");
     return MM_ERR_UNSUPPORTED;
 }
@@ -588,18 +605,20 @@ MM_EXPORT int mm_attention_sink_prefill_bf16(const void* q, const void* k_pages,
 MM_EXPORT int mm_attention_sink_decode_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, void* part_o,
                                             void* part_ml, int n_splits, const void* items,
                                             int n_items, const void* positions, const void* token_req, const void* block_table,
-                                            int table_width, int page_size, int H, int G, int dk, int dv, int window, float scale,
-                                            int sink, const void* sink_logit, const void* dist_bias, int dist_max, float softcap, int Gv,
-                                            int out_f32, void* stream) {
+                                            int table_width, int page_size, int H, int G, int dk, int dv, int window, int chunk, int keep,
+                                            float scale, int sink, const void* sink_logit, const void* dist_bias, int dist_max, float softcap, int Gv,
+                                            const void* gate, int gate_ld, int out_f32, void* stream) {
     MM_REQUIRE(Gv >= 1 && G % Gv == 0 && softcap >= 0.0f, "sink attention: the value heads must divide the key heads");
     MM_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (part_o != nullptr && part_ml != nullptr)),
                "sink attention: 1..64 splits, with scratch for more than one");
     MM_REQUIRE(n_items >= 0 && H > 0 && G > 0 && H % G == 0 && H / G <= 16, "sink attention: at most 16 query heads per kv head");
-    MM_REQUIRE(page_size > 0 && table_width > 0 && window >= 0, "sink attention: bad page geometry or window");
+    MM_REQUIRE(page_size > 0 && table_width > 0 && window >= 0 && chunk >= 0 && keep >= 0, "sink attention: bad page geometry or mask");
+    MM_REQUIRE(gate == nullptr || gate_ld >= H, "sink attention: one gate per head");
+    const KeyMask mask = {window, chunk, keep};
     if (n_items == 0) return MM_OK;
     cudaStream_t s = (cudaStream_t)stream;
     SINK_DISPATCH(launch_sink_decode, q, k_pages, v_pages, out, part_o, part_ml, n_splits, items, n_items, positions, token_req, block_table,
-                  table_width, page_size, H, G, window, scale, sink, sink_logit, dist_bias, dist_max, softcap, Gv, out_f32, s);
+                  table_width, page_size, H, G, mask, scale, sink, sink_logit, dist_bias, dist_max, softcap, Gv, gate, gate_ld, out_f32, s);
     mm_set_last_error("sink attention: key and value sizes must each be one of 32, 64, 96, 128");
     return MM_ERR_UNSUPPORTED;
 }

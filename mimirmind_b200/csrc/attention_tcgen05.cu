@@ -25,6 +25,8 @@
 // bottleneck of the whole kernel); warp 1 = MMA issuer and tensor-memory owner; warps 2..9 = softmax and output.  Same formula as the other attention kernels (reference src/compute/Attention.cpp:43-94).
 // Warp 0 requests Q and the first key tile before the CTA's set-up barrier (tensor-memory allocation, zeroing of the value
 // ring), which nothing of that needs.
+// The keys a query sees may also be its own run of tokens, and the first tokens of the sequence beside either (KeyMask): the walk over
+// key tiles then starts with the kept tokens' tiles.  A head's output may be multiplied by the logistic of a number per token.
 // All mbarrier waits are bounded; on a time-out the kernel frees its tensor memory, sets `err`
 // and returns.
 #include "tcgen05_attention.cuh"
@@ -69,7 +71,8 @@ __global__ void __launch_bounds__(ATT_TC_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                             const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out,
                             const int32_t* __restrict__ tiles, const int32_t* __restrict__ block_table, int table_width,
-                            int page_size, int H, int G, int window, float scale_log2, int sink, int* __restrict__ err) {
+                            int page_size, int H, int G, KeyMask mask, float scale_log2, int sink, const float* __restrict__ gate, int gate_ld,
+                            int* __restrict__ err) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];   // 128-byte swizzle wants 1024-byte aligned tiles
     if ((smem_u32(smem_raw) & 1023u) != 0) {                      // never seen; without the alignment nothing below is valid
         if (threadIdx.x == 0 && err != nullptr) atomicExch(err, 3);
@@ -91,8 +94,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
     const int req = tiles[tile * 4 + 0], row0 = tiles[tile * 4 + 1], n_rows = tiles[tile * 4 + 2], pos0 = tiles[tile * 4 + 3];
     const int32_t* table = block_table + (size_t)req * table_width;
     const int hi_all = pos0 + n_rows;
-    const int lo_all = (window > 0 && pos0 + 1 > window) ? pos0 + 1 - window : 0;
-    const int kt_begin = lo_all / BN, kt_end = (hi_all + BN - 1) / BN;
+    const int lo_all = mask_low(mask, pos0), keep = mask.keep;
+    const TileWalk walk = tile_walk(lo_all, keep, BN);
+    const int kt_begin = walk.begin(), kt_end = (hi_all + BN - 1) / BN;
 
     if (threadIdx.x == 64) {
         prefetch_tensormap(&tmQ);
@@ -107,8 +111,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
     // from the block table would otherwise sit, with its full latency, between every two tiles.
     auto page_of = [&](int kt) -> int {
         if (kt >= kt_end || pj >= pages_per_tile) return -1;
-        const int key_lo = kt * BN + pj * page_size;
-        return (key_lo < hi_all && key_lo + page_size > lo_all) ? table[kt * pages_per_tile + pj] : -1;
+        const int kr = walk.real(kt), key_lo = kr * BN + pj * page_size;
+        return (key_lo < hi_all && (key_lo + page_size > lo_all || key_lo < keep)) ? table[kr * pages_per_tile + pj] : -1;
     };
     constexpr int AHEAD = 4;
     int ahead[AHEAD];
@@ -241,7 +245,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
         const int row = q * 32 + lane;
         const int pos = pos0 + row;
         const bool row_valid = row < n_rows;
-        const int wlo = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+        const int wlo = mask_low(mask, pos);
         const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16);
         const uint32_t s_addr = lane_addr + g * 128, o_addr = lane_addr + 256 + g * HD;
         float m_ref = -INFINITY;           // the maximum the group's probabilities (and its O) are taken relative to
@@ -253,7 +257,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
         const SoftmaxBars bars = {smem_u32(&ctl->s_full[g]), smem_u32(&ctl->s_free[g]), smem_u32(&ctl->p_full[g]), smem_u32(&ctl->pv_done[g])};
         for (uint32_t it = g; (int)it < n_tiles_k && ok; it += 2, ++done) {
             ok = softmax_tile<HD>(bars, abort_flag, s_addr, o_addr, sP + g * TILE_BYTES, HALF_BYTES, row, lane, row_valid, pos, wlo,
-                                  (kt_begin + (int)it) * BN, it >> 1, done == 0, scale_log2, sreg, m_ref, l);
+                                  walk.real(kt_begin + (int)it) * BN, it >> 1, done == 0, scale_log2, sreg, m_ref, l, keep);
         }
         // Merge the two groups: every thread posts its row's (reference, sum); the row's output is
         // (O0 f0 + O1 f1) / (l0 f0 + l1 f1) with f = 2^((m_g - m) scale); group g writes its half of the output columns.
@@ -273,7 +277,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
         if (ok && tiles0 > 0) ok = mbar_wait(smem_u32(&ctl->pv_done[0]), (uint32_t)(tiles0 - 1) & 1, abort_flag);
         if (ok && tiles1 > 0) ok = mbar_wait(smem_u32(&ctl->pv_done[1]), (uint32_t)(tiles1 - 1) & 1, abort_flag);
         tc_fence_after();
-        const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+        const float inv = (total > 0.0f ? 1.0f / total : 0.0f) * (row_valid ? head_gate(gate, gate_ld, row0 + row, h) : 0.0f);
         __nv_bfloat16* orow = out + ((size_t)(row0 + row) * H + h) * HD + g * (HD / 2);
 #pragma unroll 1
         for (int c = 0; c < HD / 64; ++c) {                        // 32 output columns at a time
@@ -321,12 +325,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __gri
 // bounded wait ran out (may be null).
 static int attention_prefill_tcgen05_launch(const void* q, const void* k_pages, const void* v_pages, void* out,
                                             const void* tiles, int n_tiles, const void* block_table, int table_width,
-                                            int page_size, int num_pages, int n_tokens, int H, int G, int hd, int window,
-                                            float scale, int sink, void* err, void* stream) {
+                                            int page_size, int num_pages, int n_tokens, int H, int G, int hd, KeyMask mask,
+                                            float scale, int sink, const void* gate, int gate_ld, void* err, void* stream) {
     MM_REQUIRE(hd == 128 || hd == 64, "attention_prefill_tcgen05: built for head sizes 64 and 128");
     MM_REQUIRE(n_tiles >= 0 && H > 0 && G > 0 && H % G == 0 && n_tokens > 0 && num_pages > 0, "attention_prefill_tcgen05: bad sizes");
     MM_REQUIRE(page_size >= 8 && page_size <= 128 && (128 % page_size) == 0, "attention_prefill_tcgen05: page_size must be 8, 16, 32, 64 or 128");
-    MM_REQUIRE(table_width > 0 && window >= 0, "attention_prefill_tcgen05: bad table or window");
+    MM_REQUIRE(table_width > 0 && mask.window >= 0 && mask.chunk >= 0 && mask.keep >= 0, "attention_prefill_tcgen05: bad table or mask");
+    MM_REQUIRE(gate == nullptr || gate_ld >= H, "attention_prefill_tcgen05: one gate per head");
     if (n_tiles == 0) return MM_OK;
     CUtensorMap tq, tk, tv;
     const long long pool_rows = (long long)num_pages * G * page_size;
@@ -354,11 +359,11 @@ static int attention_prefill_tcgen05_launch(const void* q, const void* k_pages, 
     if (hd == 128)
         attention_prefill_tc_kernel<128><<<grid, ATT_TC_THREADS, smem, (cudaStream_t)stream>>>(
             tq, tk, tv, (__nv_bfloat16*)out, (const int32_t*)tiles, (const int32_t*)block_table, table_width, page_size, H, G,
-            window, scale * LOG2E, sink, (int*)err);
+            mask, scale * LOG2E, sink, (const float*)gate, gate_ld, (int*)err);
     else
         attention_prefill_tc_kernel<64><<<grid, ATT_TC_THREADS, smem, (cudaStream_t)stream>>>(
             tq, tk, tv, (__nv_bfloat16*)out, (const int32_t*)tiles, (const int32_t*)block_table, table_width, page_size, H, G,
-            window, scale * LOG2E, sink, (int*)err);
+            mask, scale * LOG2E, sink, (const float*)gate, gate_ld, (int*)err);
     MM_CHECK_LAUNCH();
     return MM_OK;
 }
@@ -368,15 +373,16 @@ MM_EXPORT int mm_attention_prefill_tcgen05(const void* q, const void* k_pages, c
                                            int page_size, int num_pages, int n_tokens, int H, int G, int hd, int window,
                                            float scale, void* err, void* stream) {
     return attention_prefill_tcgen05_launch(q, k_pages, v_pages, out, tiles, n_tiles, block_table, table_width, page_size, num_pages,
-                                            n_tokens, H, G, hd, window, scale, 0, err, stream);
+                                            n_tokens, H, G, hd, KeyMask{window, 0, 0}, scale, 0, nullptr, 0, err, stream);
 }
 
-// The same with a softmax sink: one is added to every row's denominator (scale must be positive).
+// The same with a softmax sink (one is added to every row's denominator; scale must be positive), any mask and a gate per head
+// (fp32 [n_tokens, gate_ld] or null).
 MM_EXPORT int mm_attention_prefill_tcgen05_sink(const void* q, const void* k_pages, const void* v_pages, void* out,
                                                 const void* tiles, int n_tiles, const void* block_table, int table_width,
-                                                int page_size, int num_pages, int n_tokens, int H, int G, int hd, int window,
-                                                float scale, int sink, void* err, void* stream) {
+                                                int page_size, int num_pages, int n_tokens, int H, int G, int hd, int window, int chunk,
+                                                int keep, float scale, int sink, const void* gate, int gate_ld, void* err, void* stream) {
     MM_REQUIRE(scale > 0.0f, "attention_prefill_tcgen05: the scale must be positive");
     return attention_prefill_tcgen05_launch(q, k_pages, v_pages, out, tiles, n_tiles, block_table, table_width, page_size, num_pages,
-                                            n_tokens, H, G, hd, window, scale, sink, err, stream);
+                                            n_tokens, H, G, hd, KeyMask{window, chunk, keep}, scale, sink, gate, gate_ld, err, stream);
 }

@@ -75,6 +75,14 @@ __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { retu
 __device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
 
+// ---- a norm without statistics, w tanh(alpha x) + b with numbers per channel ----------------------------------------------
+struct TanhNorm {
+    const float* w;     // [D] (null: no such norm)
+    const float* b;     // [D]
+    float alpha;
+};
+__device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+
 // ---- activations of one value: 0 none, 1 squared relu, 2 gelu (tanh form), 3 silu, 4 relu, 5 gelu (exact form) ----------
 #define MM_ACT_COUNT 5
 template <bool FAST>
@@ -102,6 +110,40 @@ __device__ __forceinline__ float glu_act(float g, float u, int act, float limit,
     if (act == MM_GLU_GELU_TANH) return gelu_tanh(g) * u;
     const float e = FAST ? __expf(-g) : expf(-g);
     return g / (1.0f + e) * u;
+}
+
+// ---- which keys a query sees --------------------------------------------------------------------------------------------
+// A query at position a sees a key at j <= a if it is within the last `window` tokens (0: no limit) and in the query's own run
+// of `chunk` tokens counted from position 0 (0: no runs), or if it is one of the first `keep` tokens of the sequence.
+struct KeyMask {
+    int window, chunk, keep;
+};
+// the first key of the query's own stretch (the kept first tokens aside); never falls as `pos` grows
+__host__ __device__ __forceinline__ int mask_low(const KeyMask& m, int pos) {
+    int lo = m.window > 0 && pos + 1 > m.window ? pos + 1 - m.window : 0;
+    if (m.chunk > 0) {
+        const int c = pos / m.chunk * m.chunk;
+        lo = c > lo ? c : lo;
+    }
+    return lo;
+}
+// The key tiles of a walk: those from tile `main` on, which hold the stretch, and in front of them `n_kept` tiles from the
+// sequence's start for the kept tokens.  Tiles are numbered main - n_kept .. , so the stretch's tiles keep their own numbers.
+struct TileWalk {
+    int main, n_kept;
+    __device__ __forceinline__ int begin() const { return main - n_kept; }
+    __device__ __forceinline__ int real(int t) const { return t < main ? t - (main - n_kept) : t; }
+};
+__device__ __forceinline__ TileWalk tile_walk(int lo, int keep, int tile) {
+    TileWalk w;
+    w.main = lo / tile;
+    const int k = (keep + tile - 1) / tile;
+    w.n_kept = k < w.main ? k : w.main;
+    return w;
+}
+// what a head's output is multiplied by when `gate` (fp32 [tokens, ld], null: nothing) holds its gate's projection
+__device__ __forceinline__ float head_gate(const float* gate, int ld, int t, int h) {
+    return gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-gate[(size_t)t * ld + h]));
 }
 
 // ---- reductions --------------------------------------------------------------

@@ -12,12 +12,14 @@
 // The ring is as deep as shared memory allows when the grid has at most one CTA per SM (few tiles: the bytes in
 // flight per SM are what bounds the stream), and shallow enough for two CTAs per SM otherwise.
 //
-// Epilogues, per unit of (batch row, 16 weight rows), the same four as the weight-streaming GEMV of gemv_bf16.cu
+// Epilogues, per unit of (batch row, 16 weight rows), the same as the weight-streaming GEMV of gemv_bf16.cu
 // and with the same weight layouts, so a decode layer is five launches at these batch sizes too:
 //   PLAIN   bias; fp32 or bf16 output
 //   SWIGLU  rows interleave gate and up in blocks of 8; writes silu(gate) * up
 //   RESID   adds into the fp32 residual stream; with a norm weight also writes residual * weight (bf16) and the
 //           unit's sum of squares (the next product applies 1/rms to its accumulators: `in_ss`)
+//   TANH    norms the product by w tanh(alpha x) + b, adds it into the fp32 residual stream and, with a second such norm, writes
+//           the normed sum (bf16)
 //   ROPE    q/k/v projection: bias, rotation of q and k (rows interleave each head's halves in blocks of 8), q to
 //           [M, H*hd], k and v into their cache pages
 //
@@ -42,7 +44,7 @@ constexpr int SK_BK = 64;               // k per stage: one 128-byte swizzled ro
 constexpr int SK_THREADS = 192;
 constexpr int SK_A_BYTES = SK_ROWS * SK_BK * 2;
 
-enum { SK_PLAIN = 0, SK_SWIGLU = 1, SK_RESID = 2, SK_ROPE = 3 };
+enum { SK_PLAIN = 0, SK_SWIGLU = 1, SK_RESID = 2, SK_ROPE = 3, SK_TANH = 4 };
 
 struct SkinnyArgs {
     void* out;                  // PLAIN [M, ldo] bf16/fp32; SWIGLU [M, ldo] (N/2 columns)
@@ -63,6 +65,8 @@ struct SkinnyArgs {
     __nv_bfloat16* xw_out;      // [M, N]
     float* out_ss;              // [N / 16][out_ld]
     int out_ld;
+    // TANH (with residual and xw_out)
+    TanhNorm post, next;
     // ROPE
     __nv_bfloat16* q_out;       // [M, H * hd]
     __nv_bfloat16* k_pages;     // [pages, G, page_size, hd] or null
@@ -340,6 +344,25 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
                     sk_store8_bf16(o + 8, xw + 8);
                     a.out_ss[(size_t)(n0 / 16) * a.out_ld + m] = sq;
                 }
+            } else if constexpr (EPI == SK_TANH) {
+                float* res = a.residual + (size_t)m * a.N + n0;
+#pragma unroll
+                for (int i = 0; i < 16; i += 4) {
+                    const float4 t4 = *reinterpret_cast<const float4*>(res + i);
+                    const float4 w4 = *reinterpret_cast<const float4*>(a.post.w + n0 + i), b4 = *reinterpret_cast<const float4*>(a.post.b + n0 + i);
+                    v[i] = t4.x + tanh_norm(v[i], a.post.alpha, w4.x, b4.x);
+                    v[i + 1] = t4.y + tanh_norm(v[i + 1], a.post.alpha, w4.y, b4.y);
+                    v[i + 2] = t4.z + tanh_norm(v[i + 2], a.post.alpha, w4.z, b4.z);
+                    v[i + 3] = t4.w + tanh_norm(v[i + 3], a.post.alpha, w4.w, b4.w);
+                    *reinterpret_cast<float4*>(res + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+                }
+                if (a.next.w != nullptr) {
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) v[i] = tanh_norm(v[i], a.next.alpha, a.next.w[n0 + i], a.next.b[n0 + i]);
+                    __nv_bfloat16* o = a.xw_out + (size_t)m * a.N + n0;
+                    sk_store8_bf16(o, v);
+                    sk_store8_bf16(o + 8, v + 8);
+                }
             } else {
                 const int hd = a.hd, head = n0 / hd, within = n0 - head * hd;
                 if (a.bias != nullptr) {
@@ -566,6 +589,25 @@ MM_EXPORT int mm_gemm_skinny_residual(const void* W, const void* x, void* residu
     a.residual = (float*)residual; a.norm_w = norm_w; a.norm_w_dtype = norm_w_dtype;
     a.xw_out = (__nv_bfloat16*)xw_out; a.out_ss = (float*)out_ss; a.out_ld = out_ld;
     return sk_dispatch<SK_RESID>(W, x, ldx, a, (cudaStream_t)stream);
+}
+
+// residual[M, N] (fp32) += post(x * W^T), and with next_w out[M, N] (bf16) = next(residual); a norm is w tanh(alpha v) + b with
+// fp32 numbers per column.
+MM_EXPORT int mm_gemm_skinny_tanh(const void* W, const void* x, void* residual, const void* post_w, const void* post_b, float post_alpha,
+                                  const void* next_w, const void* next_b, float next_alpha, void* out, int M, int N, int K, int ldx, int splits,
+                                  void* err, void* stream) {
+    SkinnyArgs a;
+    const int rc = sk_common(a, W, x, M, N, K, ldx, splits, nullptr, 0, 0, 0, 0.0f, err);
+    if (rc != MM_OK) return rc;
+    MM_REQUIRE(residual != nullptr && post_w != nullptr && post_b != nullptr, "gemm_skinny: no residual or no norm");
+    MM_REQUIRE((next_w == nullptr) == (next_b == nullptr) && (next_w == nullptr || out != nullptr), "gemm_skinny: a second norm needs its offset and an output");
+    MM_REQUIRE(((reinterpret_cast<uintptr_t>(residual) | reinterpret_cast<uintptr_t>(post_w) | reinterpret_cast<uintptr_t>(post_b) |
+                 reinterpret_cast<uintptr_t>(next_w) | reinterpret_cast<uintptr_t>(next_b) | reinterpret_cast<uintptr_t>(out)) & 15) == 0,
+               "gemm_skinny: residual, norms and output must be 16-byte aligned");
+    a.residual = (float*)residual; a.xw_out = (__nv_bfloat16*)out;
+    a.post = TanhNorm{(const float*)post_w, (const float*)post_b, post_alpha};
+    a.next = TanhNorm{(const float*)next_w, (const float*)next_b, next_alpha};
+    return sk_dispatch<SK_TANH>(W, x, ldx, a, (cudaStream_t)stream);
 }
 
 // q/k/v projection with bias, rotation and cache write; layouts as mm_gemv_bf16_qkv_rope.

@@ -21,6 +21,8 @@
 //           the rows of residual * weight (bf16) and, per 16-column tile, the partial sums of
 //           squares of the new residual are written too: RMSNorm(x) = (x * w) / rms(x), and the
 //           1/rms factor commutes with the next matrix product, which applies it (below).
+//   TANH    the product is normed by w tanh(alpha x) + b, added to the fp32 residual stream in place, and if a second such norm
+//           is given the normed sum is written (bf16): norms that need no other number of the row.
 //   ROPE    q/k/v projection: bias, rotary position encoding of q and k (split-half pairs; the
 //           weight rows of each q and k head interleave the two halves in blocks of 8, so a thread
 //           holds a pair), q written as [M, H * hd], k and v written into their cache pages.
@@ -57,6 +59,8 @@ struct GemvArgs {
     int norm_w_dtype;
     __nv_bfloat16* xw_out;      // [M, N]
     float* out_ss;              // [N / 16][16]
+    // TANH (with residual and xw_out)
+    TanhNorm post, next;
     // ROPE
     __nv_bfloat16* q_out;       // [M, H * hd]
     __nv_bfloat16* k_pages;     // [pages, G, page_size, hd] or null
@@ -66,7 +70,7 @@ struct GemvArgs {
     int page_size, H, G, hd;
 };
 
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_RESID = 2, EPI_ROPE = 3 };
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_RESID = 2, EPI_ROPE = 3, EPI_TANH = 4 };
 
 __device__ __forceinline__ uint4 ldg_stream(const void* p) {
     uint4 v;
@@ -158,8 +162,9 @@ __device__ __forceinline__ void gemv_item(const GemvArgs& a, int item, const Gem
     // is held and no warp waits for them before the epilogue):
     //   every EPI  the producer's partial sums of squares of the input rows, [in_tiles][M4] (dynamic shared memory)
     //   RESID      the residual values [rt][m][16 cols] and the norm weights [rt][16] of this CTA's columns
+    //   TANH       the residual values, and both norms' weights and offsets [4][rt][16] (dynamic shared memory)
     //   ROPE       cos and sin [rt][m][8] of every (row, pair) of this CTA's tiles, the bias [rt][16], each row's slot
-    constexpr bool kStaged = (EPI == EPI_RESID || EPI == EPI_ROPE);
+    constexpr bool kStaged = (EPI == EPI_RESID || EPI == EPI_ROPE || EPI == EPI_TANH);
     float* stage_a = sm.stage_a;
     float* stage_b = sm.stage_b;
     int* slot_s = sm.slot_s;
@@ -172,13 +177,13 @@ __device__ __forceinline__ void gemv_item(const GemvArgs& a, int item, const Gem
                 cp_async16(&ss_s[j * M4 + c * 4], a.in_ss + j * 16 + c * 4);
             }
         }
-        if constexpr (EPI == EPI_RESID) {
+        if constexpr (EPI == EPI_RESID || EPI == EPI_TANH) {
             for (int idx = threadIdx.x; idx < a.RT * 64; idx += GEMV_THREADS) {     // (tile, row, 4 columns)
                 const int ti = idx >> 6, m = (idx >> 2) & 15, c4 = idx & 3;
                 const int col = (item * a.RT + ti) * 16 + c4 * 4;
                 if (m < a.M && col < a.N) cp_async16(&stage_a[(ti * 16 + m) * 16 + c4 * 4], a.residual + (size_t)m * a.N + col);
             }
-            if (a.norm_w != nullptr) {
+            if (EPI == EPI_RESID && a.norm_w != nullptr) {
                 const int bytes16 = (a.norm_w_dtype == MM_F32) ? 4 : 2;             // 16-byte pieces per tile
                 for (int idx = threadIdx.x; idx < a.RT * bytes16; idx += GEMV_THREADS) {
                     const int ti = idx / bytes16, c = idx - ti * bytes16;
@@ -187,6 +192,14 @@ __device__ __forceinline__ void gemv_item(const GemvArgs& a, int item, const Gem
                         cp_async16(reinterpret_cast<char*>(&stage_b[ti * 16]) + c * 16,
                                    reinterpret_cast<const char*>(a.norm_w) + (size_t)col * (a.norm_w_dtype == MM_F32 ? 4 : 2) + c * 16);
                 }
+            }
+        }
+        if constexpr (EPI == EPI_TANH) {
+            for (int idx = threadIdx.x; idx < a.RT * 16; idx += GEMV_THREADS) {     // (vector, tile, 4 columns)
+                const int v = idx / (a.RT * 4), rest = idx - v * a.RT * 4, ti = rest >> 2, c4 = rest & 3;
+                const int col = (item * a.RT + ti) * 16 + c4 * 4;
+                const float* src = v == 0 ? a.post.w : (v == 1 ? a.post.b : (v == 2 ? a.next.w : a.next.b));
+                if (src != nullptr && col < a.N) cp_async16(&ss_s[(v * a.RT + ti) * 16 + c4 * 4], src + col);
             }
         }
         if constexpr (EPI == EPI_ROPE) {
@@ -354,6 +367,18 @@ __device__ __forceinline__ void gemv_item(const GemvArgs& a, int item, const Gem
                 sq += __shfl_xor_sync(0xffffffffu, sq, 8);
                 sq += __shfl_xor_sync(0xffffffffu, sq, 16);
                 if (live && r == 0 && a.norm_w != nullptr) a.out_ss[(n0 / 16) * 16 + m] = sq;
+            } else if constexpr (EPI == EPI_TANH) {
+                if (!live) continue;
+#pragma unroll
+                for (int hi = 0; hi < 2; ++hi) {
+                    const int c = r + hi * 8;
+                    const size_t o = (size_t)m * a.N + n0 + c;
+                    const float* nw = ss_s + rt * 16 + c;
+                    const int step = a.RT * 16;
+                    const float v = stage_a[(rt * 16 + m) * 16 + c] + tanh_norm(acc[j][hi * 2 + e], a.post.alpha, nw[0], nw[step]);
+                    a.residual[o] = v;
+                    if (a.next.w != nullptr) a.xw_out[o] = __float2bfloat16_rn(tanh_norm(v, a.next.alpha, nw[2 * step], nw[3 * step]));
+                }
             } else if constexpr (EPI == EPI_ROPE) {
                 if (!live) continue;
                 const int hd = a.hd, head = n0 / hd, within = n0 - head * hd;
@@ -423,6 +448,7 @@ MM_EXPORT int mm_set_gemv_blocks(int n) {
 }
 
 static size_t gemv_dynamic_smem(const GemvArgs& a) {
+    if (a.post.w) return (size_t)4 * a.RT * 16 * sizeof(float);                   // both norms' weights and offsets
     return a.in_ss ? (size_t)a.in_tiles * ((a.M + 3) & ~3) * sizeof(float) : 0;   // the staged partial sums of the input rows
 }
 
@@ -545,6 +571,24 @@ MM_EXPORT int mm_gemv_bf16_residual(const void* W, const void* x, void* residual
     a.residual = (float*)residual; a.norm_w = norm_w; a.norm_w_dtype = norm_w_dtype;
     a.xw_out = (__nv_bfloat16*)xw_out; a.out_ss = (float*)out_ss;
     return launch_gemv<EPI_RESID>(a, (cudaStream_t)stream);
+}
+
+// residual[M, N] (fp32) += post(x * W^T), and with next_w out[M, N] (bf16) = next(residual); a norm is w tanh(alpha v) + b with
+// fp32 numbers per column.
+MM_EXPORT int mm_gemv_bf16_tanh(const void* W, const void* x, void* residual, const void* post_w, const void* post_b, float post_alpha,
+                                const void* next_w, const void* next_b, float next_alpha, void* out, int M, int N, int K, int ldx, int rt, int ks,
+                                void* stream) {
+    GemvArgs a;
+    const int rc = gemv_common(a, W, x, M, N, K, ldx, rt, ks, nullptr, 0, 0, 0.0f);
+    if (rc != MM_OK) return rc;
+    MM_REQUIRE(residual != nullptr && post_w != nullptr && post_b != nullptr, "gemv: no residual or no norm");
+    MM_REQUIRE((next_w == nullptr) == (next_b == nullptr) && (next_w == nullptr || out != nullptr), "gemv: a second norm needs its offset and an output");
+    MM_REQUIRE(((reinterpret_cast<uintptr_t>(residual) | reinterpret_cast<uintptr_t>(post_w) | reinterpret_cast<uintptr_t>(post_b) |
+                 reinterpret_cast<uintptr_t>(next_w) | reinterpret_cast<uintptr_t>(next_b)) & 15) == 0, "gemv: residual and norms must be 16-byte aligned");
+    a.residual = (float*)residual; a.xw_out = (__nv_bfloat16*)out;
+    a.post = TanhNorm{(const float*)post_w, (const float*)post_b, post_alpha};
+    a.next = TanhNorm{(const float*)next_w, (const float*)next_b, next_alpha};
+    return launch_gemv<EPI_TANH>(a, (cudaStream_t)stream);
 }
 
 // q/k/v projection with bias, rotary encoding and cache write.  W [(H + 2G) * hd, K]: the rows of every q and k

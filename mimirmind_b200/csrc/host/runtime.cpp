@@ -7,7 +7,8 @@
 //    (src/runtime/serving/PagedKvBlockAllocator.cpp:11-60); freeing a page twice or one never given is an error;
 //  * a request has one block table per cache group, indexed by absolute position / page size; reserve is all or
 //    nothing across groups (src/runtime/serving/PagedKvSequence.cpp:41-74); tokens count after commit
-//    (src/runtime/KvCache.hpp:90-103); a windowed group gives back pages no later query can reach; release gives
+//    (src/runtime/KvCache.hpp:90-103); a group whose readers look back over a window or over their own run of
+//    tokens gives back pages no later query can reach (the kept first tokens' pages stay); release gives
 //    everything back (PagedKvSequence.cpp:76-87); every request owns a state slot (src/runtime/SsmState.hpp:39-86);
 //  * per step decodes first, then prompt portions under the token budget, in admission order
 //    (src/runtime/serving/ChunkedPrefillScheduler.cpp:20-51); first-in first-out admission up to max_active
@@ -85,6 +86,19 @@ class PageAllocator {
     long long allocs_ = 0, reuses_ = 0;
 };
 
+// Which earlier tokens a reader of a group looks at: the last `window` (0: no limit), its own run of `chunk` tokens counted from
+// position 0 (0: no runs), and always the first `keep`.
+struct ReaderMask {
+    int window = 0, chunk = 0, keep = 0;
+    bool bounded() const { return window > 0 || chunk > 0; }
+    // the first token (kept ones aside) that a query at position `pos` or later can see
+    int dead_before(int pos) const {
+        int lo = window > 0 ? std::max(0, pos + 1 - window) : 0;
+        if (chunk > 0) lo = std::max(lo, pos / chunk * chunk);
+        return lo;
+    }
+};
+
 struct CacheRequest {
     int length = 0, reserved = 0, slot = -1;
     bool started = false;
@@ -97,13 +111,29 @@ class CacheManager {
         : page_size_(page_size), slots_(max_requests) {
         for (int g = 0; g < n_groups; ++g) {
             allocs_.emplace_back(pages[g]);
-            windows_.push_back(windows[g]);
+            masks_.push_back({ReaderMask{windows[g], 0, 0}});
         }
     }
     int n_groups() const { return (int)allocs_.size(); }
     int page_size() const { return page_size_; }
     PageAllocator& allocator(int g) { return allocs_[g]; }
-    int window(int g) const { return windows_[g]; }
+    // every reader of the group looks back over a bounded stretch only
+    bool bounded(int g) const {
+        for (const ReaderMask& m : masks_[g])
+            if (!m.bounded()) return false;
+        return true;
+    }
+    int set_masks(int g, int n, const int* numbers) {
+        if (g < 0 || g >= n_groups() || n < 1) return fail("no such cache group, or no readers");
+        std::vector<ReaderMask> masks;
+        for (int i = 0; i < n; ++i) {
+            const ReaderMask m{numbers[3 * i], numbers[3 * i + 1], numbers[3 * i + 2]};
+            if (m.window < 0 || m.chunk < 0 || m.keep < 0) return fail("a reader's mask must not be negative");
+            masks.push_back(m);
+        }
+        masks_[g] = masks;
+        return 0;
+    }
     bool has(int64_t rid) const { return reqs_.count(rid) != 0; }
     CacheRequest* find(int64_t rid) {
         auto it = reqs_.find(rid);
@@ -161,14 +191,17 @@ class CacheManager {
         if (new_len < r->length || new_len > r->reserved)
             return fail("commit to " + std::to_string(new_len) + " outside [" + std::to_string(r->length) + ", " + std::to_string(r->reserved) + "]");
         r->length = new_len;
-        // the next query sits at position new_len and sees keys >= new_len + 1 - W
+        // the next query sits at position new_len: a page goes when no reader of the group can see any token of it again
         for (size_t g = 0; g < allocs_.size(); ++g) {
-            if (windows_[g] <= 0) continue;
-            const int dead_before = new_len + 1 - windows_[g];
+            int dead_before = new_len, keep = 0;
+            for (const ReaderMask& m : masks_[g]) {
+                dead_before = std::min(dead_before, m.bounded() ? m.dead_before(new_len) : 0);
+                keep = std::max(keep, m.keep);
+            }
             if (dead_before <= 0) continue;
             auto& t = r->tables[g];
             const int upto = std::min(dead_before / page_size_, (int)t.size());
-            for (int b = 0; b < upto; ++b)
+            for (int b = blocks_for(keep); b < upto; ++b)
                 if (t[b] != INVALID_PAGE) {
                     if (allocs_[g].free(t[b]) != 0) return -2;
                     t[b] = INVALID_PAGE;
@@ -220,7 +253,7 @@ class CacheManager {
   private:
     int page_size_;
     std::vector<PageAllocator> allocs_;
-    std::vector<int> windows_;
+    std::vector<std::vector<ReaderMask>> masks_;      // per group, one entry per kind of reader
     PageAllocator slots_;
     std::unordered_map<int64_t, CacheRequest> reqs_;
 };
@@ -283,7 +316,7 @@ class Scheduler {
         else {
             const int need = (n + mgr_->page_size() - 1) / mgr_->page_size();
             for (int g = 0; g < mgr_->n_groups(); ++g)
-                if (mgr_->window(g) <= 0 && need > mgr_->total_pages(g))
+                if (!mgr_->bounded(g) && need > mgr_->total_pages(g))
                     reason = "prompt needs " + std::to_string(need) + " pages, the pool has " + std::to_string(mgr_->total_pages(g));
         }
         if (!reason.empty()) {
@@ -494,6 +527,8 @@ MMH void* mmh_cache_create(int n_groups, const int* pages, const int* windows, i
     if (n_groups < 0 || page_size <= 0 || max_requests < 0) return nullptr;
     return new CacheManager(n_groups, pages, windows, page_size, max_requests);
 }
+// numbers: n triples (window, chunk, keep), one per kind of reader of the group; replaces the window it was created with
+MMH int mmh_cache_set_masks(void* h, int group, int n, const int* numbers) { return static_cast<CacheManager*>(h)->set_masks(group, n, numbers); }
 MMH void mmh_cache_destroy(void* h) { delete static_cast<CacheManager*>(h); }
 MMH int mmh_cache_has(void* h, long long rid) { return static_cast<CacheManager*>(h)->has(rid) ? 1 : 0; }
 MMH int mmh_cache_add(void* h, long long rid) { return static_cast<CacheManager*>(h)->add(rid); }

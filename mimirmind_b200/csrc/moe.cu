@@ -6,7 +6,7 @@
 //   the `keep` best runs can be chosen; of those the `top` with the largest s are taken (ties: the lower index);
 //   weights: the chosen s divided by their sum (+ 1e-20);
 //   y = sum over the chosen e of weight_e * W_down[e] (act(W_gate[e] x) * (W_up[e] x)).
-// Options: logistic scores that are not renormed; a correction per expert added to the scores for the choice only; runs
+// Options: logistic scores, as they are or renormed like the others; a factor on the weights; a correction per expert added to the scores for the choice only; runs
 // scored by the sum of their two best choice scores; experts of two matrices, W_down[e] act(W_up[e] x); one more row of the
 // router's matrix whose logistic value gates something else per token.
 //
@@ -32,12 +32,12 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {      // the larg
 }
 
 // One warp: the choice for one token from its E logits `zr`; scratch: 2 E + 2 groups floats of the warp's own.
-// scoring 0: s = softmax(z), the chosen weights divided by their sum; 1: s = sigmoid(z), the chosen weights as they are.
+// scoring 0: s = softmax(z); 1: s = sigmoid(z).  renorm: the chosen weights are divided by their sum; then all are multiplied by wscale.
 // The choice goes by c = s + correction (null: c = s), which may be negative; a run of experts is scored by its best c, or
 // with pair_sum by the sum of its two best (a run of one: its only one).
 __device__ __forceinline__ void moe_route_warp(const float* zr, float* scratch, int lane, int E, int top, int groups, int keep,
                                                int32_t* __restrict__ idx, float* __restrict__ wts, size_t t, int scoring = 0,
-                                               const float* __restrict__ correction = nullptr, int pair_sum = 0) {
+                                               const float* __restrict__ correction = nullptr, int pair_sum = 0, int renorm = 1, float wscale = 1.0f) {
     float* s = scratch;
     float* c = scratch + E;
     float* gs = scratch + 2 * E;
@@ -112,9 +112,9 @@ __device__ __forceinline__ void moe_route_warp(const float* zr, float* scratch, 
         }
     }
     __syncwarp();
-    if (lane == 0 && scoring == 0) {
-        const float d = total + 1e-20f;
-        for (int kk = 0; kk < top; ++kk) wts[t * top + kk] /= d;
+    if (lane == 0 && (renorm || wscale != 1.0f)) {
+        const float d = renorm ? total + 1e-20f : 1.0f;
+        for (int kk = 0; kk < top; ++kk) wts[t * top + kk] = wts[t * top + kk] / d * wscale;
     }
 }
 
@@ -153,7 +153,7 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
 template <typename T, int TOK>
 __global__ void __launch_bounds__(1024) moe_router_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, int n_tokens, int D, int E, int top,
                                                          int groups, int keep, int vec, int32_t* __restrict__ idx, float* __restrict__ wts, int scoring,
-                                                         const float* __restrict__ correction, int pair_sum, float* __restrict__ gate) {
+                                                         const float* __restrict__ correction, int pair_sum, float* __restrict__ gate, int renorm, float wscale) {
     extern __shared__ float route_smem[];      // per token: logits [E + 1], then the choice's scratch [2 E + 2 groups]
     const int rows = gate ? E + 1 : E;         // with a gate the matrix has one more row, for it
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
@@ -204,15 +204,16 @@ __global__ void __launch_bounds__(1024) moe_router_kernel(const T* __restrict__ 
         if (t >= (size_t)n_tokens) break;
         float* mine = route_smem + k * per_token;
         if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-mine[E]));
-        moe_route_warp(mine, mine + E + 1, lane, E, top, groups, keep, idx, wts, t, scoring, correction, pair_sum);
+        moe_route_warp(mine, mine + E + 1, lane, E, top, groups, keep, idx, wts, t, scoring, correction, pair_sum, renorm, wscale);
     }
 }
 
 // w fp32 [E, D], or [E + 1, D] with `gate` (fp32 [n_tokens]), which gets the logistic of the last row's product;
 // correction fp32 [E] or null
 MM_EXPORT int mm_moe_router_choice(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,
-                                   int scoring, const void* correction, int pair_sum, void* gate, void* idx, void* wts, void* stream) {
-    MM_REQUIRE(scoring == 0 || scoring == 1, "moe router: the scoring is 0 (softmax, renormed) or 1 (sigmoid, as it is)");
+                                   int scoring, const void* correction, int pair_sum, void* gate, int renorm, float wscale, void* idx, void* wts,
+                                   void* stream) {
+    MM_REQUIRE(scoring == 0 || scoring == 1, "moe router: the scoring is 0 (softmax) or 1 (sigmoid)");
     MM_REQUIRE(n_tokens >= 0 && D > 0 && ldx >= D && E > 0 && top > 0 && top <= E && groups > 0 && E % groups == 0 && keep > 0 && keep <= groups,
                "moe router: experts must split into equal runs, and 0 < top <= experts, 0 < keep <= runs");
     const size_t per_token = (size_t)(3 * E + 1 + 2 * groups) * sizeof(float);
@@ -227,11 +228,11 @@ MM_EXPORT int mm_moe_router_choice(const void* x, int x_dtype, int ldx, const vo
     const int vec = D % 8 == 0 && ldx % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
     if (x_dtype == MM_F32)
         mm_launch(tok == 4 ? moe_router_kernel<float, 4> : moe_router_kernel<float, 1>, blocks, dim3(threads), smem, (cudaStream_t)stream, (const float*)x, ldx,
-                  (const float*)w, n_tokens, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate);
+                  (const float*)w, n_tokens, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring, (const float*)correction, pair_sum, (float*)gate, renorm, wscale);
     else if (x_dtype == MM_BF16)
         mm_launch(tok == 4 ? moe_router_kernel<__nv_bfloat16, 4> : moe_router_kernel<__nv_bfloat16, 1>, blocks, dim3(threads), smem, (cudaStream_t)stream,
                   (const __nv_bfloat16*)x, ldx, (const float*)w, n_tokens, D, E, top, groups, keep, vec, (int32_t*)idx, (float*)wts, scoring,
-                  (const float*)correction, pair_sum, (float*)gate);
+                  (const float*)correction, pair_sum, (float*)gate, renorm, wscale);
     else
         MM_REQUIRE(false, "moe router: dtype must be float32 or bfloat16");
     MM_CHECK_LAUNCH();
@@ -240,7 +241,7 @@ MM_EXPORT int mm_moe_router_choice(const void* x, int x_dtype, int ldx, const vo
 
 MM_EXPORT int mm_moe_router_scored(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,
                                    int scoring, void* idx, void* wts, void* stream) {
-    return mm_moe_router_choice(x, x_dtype, ldx, w, n_tokens, D, E, top, groups, keep, scoring, nullptr, 0, nullptr, idx, wts, stream);
+    return mm_moe_router_choice(x, x_dtype, ldx, w, n_tokens, D, E, top, groups, keep, scoring, nullptr, 0, nullptr, scoring == 0, 1.0f, idx, wts, stream);
 }
 
 MM_EXPORT int mm_moe_router(const void* x, int x_dtype, int ldx, const void* w, int n_tokens, int D, int E, int top, int groups, int keep,

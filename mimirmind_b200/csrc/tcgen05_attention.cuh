@@ -61,11 +61,12 @@ struct SoftmaxBars {
 
 // One thread's row of one tile of 128 keys, the group's tile number `u` (`first`: its first): S from tensor memory into `sreg`,
 // masked by position, O (O_COLS columns at o_addr) rescaled when the row's maximum has outgrown its reference by RESCALE_STEP,
-// P rounded to bf16 into p_tile (two halves of 64 keys, 128-byte swizzle), the row's sum added to l.  False: a wait ran out.
+// P rounded to bf16 into p_tile (two halves of 64 keys, 128-byte swizzle), the row's sum added to l.  The row sees keys wlo .. pos and
+// the first `keep` ones.  False: a wait ran out.
 template <int O_COLS>
 __device__ __forceinline__ bool softmax_tile(const SoftmaxBars& bars, volatile int* abort_flag, uint32_t s_addr, uint32_t o_addr, unsigned char* p_tile,
                                              uint32_t half_bytes, int row, int lane, bool row_valid, int pos, int wlo, int key0, uint32_t u, bool first,
-                                             float scale_log2, uint32_t (&sreg)[128], float& m_ref, float& l) {
+                                             float scale_log2, uint32_t (&sreg)[128], float& m_ref, float& l, int keep = 0) {
     constexpr int BN = 128;
     if (!mbar_wait(bars.s_full, u & 1, abort_flag)) return false;
     tc_fence_after();
@@ -80,6 +81,13 @@ __device__ __forceinline__ bool softmax_tile(const SoftmaxBars& bars, volatile i
     if (interior) {
 #pragma unroll
         for (int i = 0; i < BN; ++i) mx = fmaxf(mx, __uint_as_float(sreg[i]));
+    } else if (key0 < keep) {                      // a tile with kept tokens (uniform over the CTA)
+#pragma unroll
+        for (int i = 0; i < BN; ++i) {
+            const int key = key0 + i;
+            if (!(row_valid && key <= pos && (key >= wlo || key < keep))) sreg[i] = 0xff800000u;
+            mx = fmaxf(mx, __uint_as_float(sreg[i]));
+        }
     } else {
 #pragma unroll
         for (int i = 0; i < BN; ++i) {

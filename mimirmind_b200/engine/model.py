@@ -53,13 +53,11 @@ class Model:
                        [(a.name, tuple(a.shape), a.dtype) for a in theirs.token_arrays()]
                 if not same:
                     raise ValueError(f"schedule entry {i} reads the cache of entry {e.cache_from}, whose per-token arrays differ from its own")
-                if theirs.window and (not mine.window or mine.window > theirs.window):
-                    raise ValueError(f"schedule entry {i} looks back {mine.window or 'over all'} tokens, entry {e.cache_from} keeps only "
-                                     f"the last {theirs.window}")
 
     # ---- what the cache has to hold --------------------------------------------
     def cache_groups(self) -> List[GroupSpec]:
-        """Schedule entries that own a paged cache, grouped by what they keep per token and how far back they look."""
+        """Schedule entries that own a paged cache, grouped by what they keep per token and which earlier tokens they, and the
+        entries that read their cache, look at."""
         by_key: Dict[tuple, List[int]] = {}
         for i, e in enumerate(self.schedule):
             if e.cache_from is not None:
@@ -71,14 +69,20 @@ class Model:
                            for a in ks.token_arrays())
             if any(len(shape) < 1 or min(shape) < 1 for _n, shape, _d in arrays) or len({n for n, _s, _d in arrays}) != len(arrays):
                 raise ValueError(f"schedule entry {i}: per-token cache arrays need distinct names and at least one axis of positive sizes")
-            by_key.setdefault((ks.num_kv_heads, ks.head_dim, ks.window, arrays if ks.arrays else ()), []).append(i)
+            readers = [self.layers[o.layer].mixer.kv_cache_spec() for o in self.schedule if o.cache_from == i]
+            masks = tuple(sorted({m.mask() for m in [ks] + readers}))
+            if (0, 0, 0) in masks:
+                masks = ((0, 0, 0),)
+            by_key.setdefault((ks.num_kv_heads, ks.head_dim, masks, arrays if ks.arrays else ()), []).append(i)
         groups = []
-        for (g, hd, w, arrays), entries in by_key.items():
+        for (g, hd, masks, arrays), entries in by_key.items():
             if arrays:
                 name = "cache_" + "_".join(n + "x".join(str(x) for x in shape) for n, shape, _d in arrays)
             else:
                 name = f"kv{g}x{hd}"
-            groups.append(GroupSpec(name + (f"_w{w}" if w else "_full"), tuple(entries), g, hd, w, arrays))
+            name += "".join("_" + "".join(f"{letter}{x}" for letter, x in zip("wck", m) if x) for m in masks) if masks != ((0, 0, 0),) else "_full"
+            window = max(m[0] for m in masks) if all(m[0] and not m[1] for m in masks) else 0
+            groups.append(GroupSpec(name, tuple(entries), g, hd, window, arrays, masks))
         return groups
 
     EMBEDDING_STATE = -1      # the key of the embedding's state among the schedule entries' (which count from 0)

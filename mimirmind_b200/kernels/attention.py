@@ -41,10 +41,10 @@ def _sink_lib():
     if not _sink_declared:
         P, I, F = c_void_p, c_int, c_float
         _lib.declare("mm_attention_sink_supported", [I, I])
-        _lib.declare("mm_attention_sink_prefill_bf16", [P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, P, P, I, F, I, I, P])
-        _lib.declare("mm_attention_sink_decode_bf16", [P, P, P, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, P, I, F, I, I, P])
-        _lib.declare("mm_attention_decode_tma_bf16_sink", [P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, I, P, P])
-        _lib.declare("mm_attention_prefill_tcgen05_sink", [P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, F, I, P, P])
+        _lib.declare("mm_attention_sink_prefill_bf16", [P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, F, I, P, P, I, F, I, P, I, I, P])
+        _lib.declare("mm_attention_sink_decode_bf16", [P, P, P, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P, I, F, I, P, I, I, P])
+        _lib.declare("mm_attention_decode_tma_bf16_sink", [P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, I, P, I, P, P])
+        _lib.declare("mm_attention_prefill_tcgen05_sink", [P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, F, I, P, I, P, P])
         _sink_declared = True
     return _lib.load()
 
@@ -53,12 +53,17 @@ SINK_TARGET_CTAS = 2 * 148     # decode CTAs wanted: the key tiles of a token ar
 SINK_MAX_SPLITS = 16
 
 
-def sink_splits(n_items: int, num_kv_heads: int, window: int, max_kv_len: int) -> int:
+def visible_keys(window: int, chunk: int, keep: int, max_kv_len: int) -> int:
+    """The most keys a query of a step sees."""
+    limits = [n for n in (window, chunk) if n > 0]
+    return min(min(limits) + keep, max_kv_len) if limits else max_kv_len
+
+
+def sink_splits(n_items: int, num_kv_heads: int, keys: int) -> int:
     """CTAs per (token, KV head) of the decode kernel: enough to fill the GPU, never more than the token has key tiles."""
     ctas = max(1, n_items * num_kv_heads)
     if ctas >= SINK_TARGET_CTAS // 2:
         return 1
-    keys = min(window, max_kv_len) if window > 0 else max_kv_len
     return max(1, min(-(-SINK_TARGET_CTAS // ctas), -(-keys // 64), SINK_MAX_SPLITS))
 
 
@@ -97,7 +102,7 @@ def sink_plan(ctx, n_tokens: int, tile_rows: int = SINK_TILE_ROWS):
 
 def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, window: int,
                          scale: float, sink: bool, sink_logit=None, dist_bias=None, softcap: float = 0.0, value_heads=None,
-                         k_pages=None, v_pages=None, value_row=None) -> torch.Tensor:
+                         k_pages=None, v_pages=None, value_row=None, chunk: int = 0, keep: int = 0, gate=None) -> torch.Tensor:
     """Windowed attention with a softmax sink over pools of keys ``[pages, G, page, key_dim]`` and values
     ``[pages, G, page, value_dim]``.  bfloat16 with key and value sizes the tensor-core kernels are built for: a tiled
     kernel for portions, a kernel that shares keys between the query heads of a KV head for single tokens; anything
@@ -107,6 +112,8 @@ def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, 
     the value pool has that many heads and key head ``g`` reads value head ``g mod value_heads`` (several key heads over one
     set of values).  ``k_pages`` / ``v_pages``: the pools, if they are not the cache's arrays ``k`` and ``v``; ``value_row``:
     how many numbers lie between the values of consecutive tokens (values that are a slice of a wider per-token array).
+    ``chunk`` > 0: a query sees only keys of its own run of that many tokens, counted from position 0; ``keep``: the first ``keep``
+    tokens are seen whatever the window or the run; ``gate`` (fp32 [n, >= heads]): head outputs are multiplied by its logistic.
     ``out`` may be fp32 beside bfloat16 queries: the result is then not rounded (what follows takes a difference of heads)."""
     table = cache.block_table
     k_pages = cache.arrays["k"] if k_pages is None else k_pages
@@ -125,6 +132,7 @@ def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, 
         sink_ptr = sink_logit.data_ptr() if sink_logit is not None else None
         bias_ptr = dist_bias.data_ptr() if dist_bias is not None else None
         dist_max = dist_bias.shape[1] - 1 if dist_bias is not None else 0
+        gate_ptr, gate_ld = ops.gate_args(gate, q.shape[0], num_heads)
         tensor_memory = (USE_SINK_TCGEN05 and not extended and key_dim == value_dim
                          and attention_bf16.tcgen05_prefill_usable(key_dim, cache.page_size))
         tiles, n_tiles, items, n_items = sink_plan(ctx, q.shape[0], attention_bf16.TILE_ROWS_TC if tensor_memory else SINK_TILE_ROWS)
@@ -132,20 +140,20 @@ def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, 
         if n_tiles and tensor_memory:
             check(lib.mm_attention_prefill_tcgen05_sink(q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), tiles.data_ptr(),
                                                         n_tiles, table.data_ptr(), table.shape[1], cache.page_size, k_pages.shape[0],
-                                                        q.shape[0], num_heads, num_kv_heads, key_dim, int(window), float(scale),
-                                                        int(bool(sink)), ops.tcgen05_error_flag(q.device).data_ptr(), stream),
+                                                        q.shape[0], num_heads, num_kv_heads, key_dim, int(window), int(chunk), int(keep), float(scale),
+                                                        int(bool(sink)), gate_ptr, gate_ld, ops.tcgen05_error_flag(q.device).data_ptr(), stream),
                   "attention_prefill_tcgen05_sink")
         elif n_tiles:
             check(lib.mm_attention_sink_prefill_bf16(q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), tiles.data_ptr(),
                                                      n_tiles, table.data_ptr(), table.shape[1], cache.page_size, num_heads, num_kv_heads,
-                                                     key_dim, value_dim, int(window), float(scale), int(bool(sink)), sink_ptr, bias_ptr, dist_max,
-                                                     float(softcap), value_heads, out_f32, stream),
+                                                     key_dim, value_dim, int(window), int(chunk), int(keep), float(scale), int(bool(sink)), sink_ptr, bias_ptr,
+                                                     dist_max, float(softcap), value_heads, gate_ptr, gate_ld, out_f32, stream),
                   "attention_sink_prefill_bf16")
         tma = None
         if n_items and USE_SINK_TMA_DECODE and not extended and key_dim == value_dim and key_dim in (64, 128) and cache.page_size in (8, 16, 32, 64):
             # equal key and value sizes of 64 or 128: the TMA decode kernel of the plain attention, in the forms that
             # finish a row inside the kernel (one split, or the splits of a token as one cluster)
-            keys = min(window, ctx.max_kv_len) if window > 0 else ctx.max_kv_len
+            keys = visible_keys(window, chunk, keep, ctx.max_kv_len)
             _len, max_splits, cluster = attention_bf16.choose_split(n_items, num_kv_heads, keys, key_dim, cache.page_size)
             if cluster or max_splits == 1:
                 tma = (max_splits, cluster)
@@ -153,11 +161,11 @@ def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, 
             check(lib.mm_attention_decode_tma_bf16_sink(q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
                                                         items.data_ptr() if items is not None else None, n_items, ctx.positions.data_ptr(),
                                                         ctx.token_req.data_ptr(), table.data_ptr(), table.shape[1], cache.page_size,
-                                                        k_pages.shape[0], num_heads, num_kv_heads, key_dim, int(window), float(scale),
-                                                        tma[0], int(tma[1]), int(bool(sink)), ops.tcgen05_error_flag(q.device).data_ptr(), stream),
+                                                        k_pages.shape[0], num_heads, num_kv_heads, key_dim, int(window), int(chunk), int(keep), float(scale),
+                                                        tma[0], int(tma[1]), int(bool(sink)), gate_ptr, gate_ld, ops.tcgen05_error_flag(q.device).data_ptr(), stream),
                   "attention_decode_tma_bf16_sink")
         elif n_items:
-            splits = sink_splits(n_items, num_kv_heads, window, ctx.max_kv_len)
+            splits = sink_splits(n_items, num_kv_heads, visible_keys(window, chunk, keep, ctx.max_kv_len))
             part_o = part_ml = None
             if splits > 1:
                 skey = ("sink_attention_scratch", n_items, num_heads, splits, value_dim)
@@ -170,13 +178,13 @@ def paged_sink_attention(q, cache, out, ctx, num_heads: int, num_kv_heads: int, 
                                                     part_ml.data_ptr() if part_ml is not None else None, splits,
                                                     items.data_ptr() if items is not None else None, n_items, ctx.positions.data_ptr(),
                                                     ctx.token_req.data_ptr(), table.data_ptr(), table.shape[1], cache.page_size, num_heads,
-                                                    num_kv_heads, key_dim, value_dim, int(window), float(scale), int(bool(sink)), sink_ptr, bias_ptr,
-                                                    dist_max, float(softcap), value_heads, out_f32, stream),
+                                                    num_kv_heads, key_dim, value_dim, int(window), int(chunk), int(keep), float(scale), int(bool(sink)), sink_ptr,
+                                                    bias_ptr, dist_max, float(softcap), value_heads, gate_ptr, gate_ld, out_f32, stream),
                   "attention_sink_decode_bf16")
         return out
     return ops.attention_sink_generic(q, k_pages, v_pages, out, ctx.positions, ctx.token_req, table, cache.page_size, num_heads,
                                       num_kv_heads, key_dim, value_dim, window, scale, sink, sink_logit=sink_logit, dist_bias=dist_bias,
-                                      softcap=softcap, value_heads=value_heads, value_row=value_row)
+                                      softcap=softcap, value_heads=value_heads, value_row=value_row, chunk=chunk, keep=keep, gate=gate)
 
 
 USE_LATENT_MMA = True      # False: the latent attention always runs the fp32-arithmetic kernel (tests compare the two)

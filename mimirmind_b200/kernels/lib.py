@@ -59,7 +59,7 @@ _PROTOTYPES = {
     "mm_embedding_bigram": [P, P, P, P, P, P, P, P, I, P, I, I, I, I, c_longlong, c_longlong, P],
     "mm_qkv_pairs_post": [P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, P],
     "mm_rope_pairs_table": [P, P, P, I, I, P],
-    "mm_attention_sink_generic": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P, I, F, I, I, I, P],
+    "mm_attention_sink_generic": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, I, F, I, I, P, I, I, P],
     "mm_mingru_walk": [P, P, I, P, P, P, P, P, I, I, P],
     "mm_mingru_chunked": [P, P, I, P, P, P, P, P, P, P, P, I, I, I, P],
     "mm_bias_act": [P, P, I, P, I, I, I, I, P],
@@ -85,7 +85,12 @@ _PROTOTYPES = {
     "mm_head_matmul": [P, c_longlong, I, P, P, c_longlong, I, I, I, I, I, I, P],
     "mm_head_finish": [P, I, I, F, I, F, F, P, I, P, I, I, I, I, I, P],
     "mm_moe_router_scored": [P, I, I, P, I, I, I, I, I, I, I, P, P, P],
-    "mm_moe_router_choice": [P, I, I, P, I, I, I, I, I, I, I, P, I, P, P, P, P],
+    "mm_moe_router_choice": [P, I, I, P, I, I, I, I, I, I, I, P, I, P, I, F, P, P, P],
+    "mm_qk_prep": [P, I, I, I, I, I, P, P, F, P, I, I, P, P, P, I, P, I, I, I, I, I, I, P],
+    "mm_tanh_norm_chain": [P, P, I, P, P, I, P, P, F, P, P, F, P, P, I, I, I, P],
+    "mm_gemv_bf16_tanh": [P, P, P, P, P, F, P, P, F, P, I, I, I, I, I, I, P],
+    "mm_gemm_skinny_tanh": [P, P, P, P, P, F, P, P, F, P, I, I, I, I, I, P, P],
+    "mm_soft_cap": [P, c_longlong, F, P],
     "mm_moe_gemm_act": [P, I, I, P, I, P, I, I, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
     "mm_gemm_tcgen05_grouped_act": [P, P, P, I, I, I, I, I, I, I, P, P, I, I, F, P, P],
     "mm_moe_gather_scaled": [P, I, P, P, P, P, I, I, P],

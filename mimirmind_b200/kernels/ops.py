@@ -379,6 +379,37 @@ def gemv_bf16_residual(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor,
     return None if norm_weight is None else (xw, RowScale(ss, n, float(eps)))
 
 
+def gemv_tanh_supported(rt, w: torch.Tensor, m: int) -> bool:
+    """True if a step's last product over ``m`` rows and the matrix ``w`` can norm, add and norm in its epilogue (gemv_bf16_tanh)."""
+    return rt.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and rt.matmul != "simt" and small_batch_supported(m, w.shape[0], w.shape[1])
+
+
+def gemv_bf16_tanh(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor, post, then=None) -> Optional[torch.Tensor]:
+    """residual[M, N] (fp32, in place) += post(x @ w^T); with ``then`` returns then(residual) in bfloat16.  A norm is (weight,
+    offset, alpha), ``weight tanh(alpha v) + offset`` with fp32 numbers per column."""
+    _need(x, "gemv x", torch.bfloat16)
+    _need(w, "gemv w", torch.bfloat16)
+    _need(residual, "gemv residual", torch.float32)
+    m, k = x.shape
+    n = w.shape[0]
+    if w.shape != (n, k) or residual.shape != (m, n) or not small_batch_supported(m, n, k):
+        raise KernelError(f"gemv tanh: shapes x{tuple(x.shape)} w{tuple(w.shape)} residual{tuple(residual.shape)} are not supported")
+    for norm in (post, then):
+        for t in norm[:2] if norm is not None else ():
+            _need(t, "norm", torch.float32)
+            if t.shape != (n,):
+                raise KernelError("gemv tanh: weight and offset have one number per column")
+    out = torch.empty((m, n), dtype=torch.bfloat16, device=x.device) if then is not None else None
+    q = then or (None, None, 0.0)
+    common = (w.data_ptr(), x.data_ptr(), residual.data_ptr(), post[0].data_ptr(), post[1].data_ptr(), float(post[2]), _ptr(q[0]), _ptr(q[1]), float(q[2]),
+              _ptr(out), m, n, k, k)
+    if m > GEMV_MAX_ROWS:
+        check(_lib.load().mm_gemm_skinny_tanh(*common, _skinny_splits(n, k), tcgen05_error_flag(x.device).data_ptr(), _stream()), "gemm_skinny_tanh")
+    else:
+        check(_lib.load().mm_gemv_bf16_tanh(*common, *_gemv_layout(n, k), _stream()), "gemv_bf16_tanh")
+    return out
+
+
 def interleave_halves(t: torch.Tensor, num_rot_heads: int, head_dim: int) -> torch.Tensor:
     """Row order the fused q/k/v product wants: within each of the first ``num_rot_heads`` heads (q and k), rows
     16b..16b+7 are elements 8b.. of the head's first half and rows 16b+8..16b+15 the same elements of the second
@@ -748,18 +779,31 @@ def qkv_pairs_post(qkv: torch.Tensor, q_out: torch.Tensor, k_pages: Optional[tor
                                         page_size, n, H, G, dk, dv, int(rot_dims), int(mix_mode), float(mix), _stream()), "qkv_pairs_post")
 
 
+def gate_args(gate: Optional[torch.Tensor], n: int, heads: int):
+    """(pointer, row stride) of a gate per token and head for the attention kernels."""
+    if gate is None:
+        return None, 0
+    if gate.dtype != torch.float32 or not gate.is_cuda or gate.stride(1) != 1 or gate.shape[0] != n or gate.shape[1] < heads:
+        raise KernelError("attention: the gate is fp32 [n, heads] with unit column stride")
+    return gate.data_ptr(), gate.stride(0)
+
+
 def attention_sink_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,
                            token_req: torch.Tensor, block_table: torch.Tensor, page_size: int, num_heads: int, num_kv_heads: int,
                            key_dim: int, value_dim: int, window: int, scale: float, sink: bool,
                            sink_logit: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                           value_heads: Optional[int] = None, value_row: Optional[int] = None) -> torch.Tensor:
+                           value_heads: Optional[int] = None, value_row: Optional[int] = None, chunk: int = 0, keep: int = 0,
+                           gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Windowed causal attention of every token over its request's pages with keys of ``key_dim`` and values of
     ``value_dim``; with ``sink`` the softmax denominator has one added, with ``sink_logit`` (fp32 [heads]) the head's
     ``exp(logit)``; ``dist_bias`` (fp32 [heads, distances]) is added to the scaled score by distance, a head's last entry
     standing for every larger distance (fp32 arithmetic, any sizes).  ``softcap`` > 0: the scaled score becomes
     ``cap * tanh(score / cap)``.  ``value_heads``: heads of the value pool (key head g reads value head g mod value_heads);
     ``value_row``: numbers between the values of consecutive tokens (default ``value_dim``; larger when the values are the
-    leading part of a wider per-token array, which may be the key pool itself).  ``out`` has q's type or is fp32."""
+    leading part of a wider per-token array, which may be the key pool itself).  ``chunk`` > 0: a query sees only its own run of
+    ``chunk`` tokens (counted from position 0); ``keep``: the sequence's first ``keep`` tokens are seen whatever the window or run;
+    ``gate`` (fp32 [n, >= heads], may be a column slice): a head's output is multiplied by the logistic of its number.
+    ``out`` has q's type or is fp32."""
     value_heads = num_kv_heads if value_heads is None else int(value_heads)
     value_row = value_dim if value_row is None else int(value_row)
     _need(q, "attention q")
@@ -785,9 +829,9 @@ def attention_sink_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
     check(_lib.load().mm_attention_sink_generic(
         q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), dtype_code(q.dtype), positions.data_ptr(),
         token_req.data_ptr(), block_table.data_ptr(), block_table.shape[1], page_size, n, num_heads, num_kv_heads, key_dim,
-        value_dim, int(window), float(scale), int(bool(sink)), _ptr(sink_logit), _ptr(dist_bias),
+        value_dim, int(window), int(chunk), int(keep), float(scale), int(bool(sink)), _ptr(sink_logit), _ptr(dist_bias),
         dist_bias.shape[1] - 1 if dist_bias is not None else 0, float(softcap), value_heads, value_row,
-        int(out.dtype == torch.float32 and q.dtype != torch.float32), _stream()), "attention_sink_generic")
+        *gate_args(gate, n, num_heads), int(out.dtype == torch.float32 and q.dtype != torch.float32), _stream()), "attention_sink_generic")
     return out
 
 
@@ -1135,10 +1179,11 @@ GROUP_SCORES = {"max": 0, "top2_sum": 1}
 
 
 def moe_router(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: int, scoring: str = "softmax",
-               correction: Optional[torch.Tensor] = None, group_score: str = "max", gate: bool = False):
+               correction: Optional[torch.Tensor] = None, group_score: str = "max", gate: bool = False, renorm: Optional[bool] = None,
+               scale: float = 1.0):
     """The router's product (fp32 sums over ``x`` [n, D] and the fp32 matrix ``w`` [E, D]) and its choice in one launch:
-    (experts int32 [n, top], weights fp32 [n, top]).  ``scoring``: ``softmax`` (the chosen scores divided by their sum) or
-    ``sigmoid`` (the chosen scores as they are).  ``correction`` fp32 [E] is added to the scores for the choice only;
+    (experts int32 [n, top], weights fp32 [n, top]).  ``scoring``: ``softmax`` or ``sigmoid``; ``renorm``: the chosen scores are
+    divided by their sum (None: those of a softmax are, logistic ones are taken as they are); ``scale`` multiplies the weights.  ``correction`` fp32 [E] is added to the scores for the choice only;
     ``group_score``: a run of experts counts by its best choice score, or by the sum of its two best.  With ``gate`` the matrix
     has one more row, whose product's logistic value comes back as a third result, fp32 [n]."""
     _need(x, "router rows")
@@ -1155,8 +1200,9 @@ def moe_router(x: torch.Tensor, w: torch.Tensor, top: int, groups: int, keep: in
     idx = torch.empty((n, top), dtype=torch.int32, device=x.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=x.device)
     check(_lib.load().mm_moe_router_choice(x.data_ptr(), dtype_code(x.dtype), D, w.data_ptr(), n, D, E, int(top), int(groups), int(keep),
-                                           ROUTER_SCORINGS[scoring], _ptr(correction), GROUP_SCORES[group_score], _ptr(gates), idx.data_ptr(),
-                                           wts.data_ptr(), _stream()), "moe_router")
+                                           ROUTER_SCORINGS[scoring], _ptr(correction), GROUP_SCORES[group_score], _ptr(gates),
+                                           int(scoring == "softmax" if renorm is None else renorm), float(scale), idx.data_ptr(), wts.data_ptr(),
+                                           _stream()), "moe_router")
     return (idx, wts, gates) if gate else (idx, wts)
 
 
@@ -1733,3 +1779,93 @@ def scaled_sum2(a: torch.Tensor, b: torch.Tensor, ca: float, cb: float, gate: Op
                                      a.shape[-1], _stream()),
           "scaled_sum2")
     return out
+
+
+# ---- norms without statistics (csrc/norm_tanh.cu) ------------------------------------------------------------------------------
+def tanh_norm_chain(residual: torch.Tensor, branch: Optional[torch.Tensor], post, then, out: Optional[torch.Tensor] = None, *,
+                    rows: Optional[torch.Tensor] = None, wts: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """With a ``branch``: ``residual`` [n, D] (fp32, in place) gets ``post(branch)`` added (``post`` None: the branch itself).  With
+    ``then``: ``out`` [n, D] = ``then(residual)``.  A norm is (weight, offset, alpha): ``w tanh(alpha x) + b``, fp32 [D] each.  The
+    branch may be the chosen experts' rows [n * top, D] with their weights ``wts`` fp32 [n, top] and, in sorted order, their
+    ``place``.  With ``rows`` (no branch) only those rows of the residual are read."""
+    _need(residual, "residual", torch.float32)
+    D = residual.shape[1]
+    n = residual.shape[0] if rows is None else rows.numel()
+    for norm in (post, then):
+        if norm is not None:
+            for t in norm[:2]:
+                _need(t, "norm weight", torch.float32)
+                if t.shape != (D,):
+                    raise KernelError("tanh norm: weight and offset have one number per channel")
+    top = 0
+    if branch is not None:
+        _need(branch, "branch")
+        if rows is not None:
+            raise KernelError("tanh norm: a gathered call adds nothing")
+        if wts is not None:
+            _need(wts, "branch weights", torch.float32)
+            top = wts.shape[1]
+            if wts.shape[0] != n or branch.shape != (n * top, D):
+                raise KernelError("tanh norm: shape mismatch of the chosen rows")
+            if place is not None:
+                _need(place, "places", torch.int32)
+        elif branch.shape != (n, D):
+            raise KernelError("tanh norm: shape mismatch")
+    if then is not None:
+        _need(out, "tanh norm out")
+        if out.shape != (n, D):
+            raise KernelError("tanh norm: out has another shape")
+    p, q = post or (None, None, 0.0), then or (None, None, 0.0)
+    check(_lib.load().mm_tanh_norm_chain(residual.data_ptr(), _ptr(branch), dtype_code(branch.dtype) if branch is not None else F32, _ptr(wts), _ptr(place), top,
+                                         _ptr(p[0]), _ptr(p[1]), float(p[2]), _ptr(q[0]), _ptr(q[1]), float(q[2]), _ptr(rows),
+                                         _ptr(out) if then is not None else None, dtype_code(out.dtype) if then is not None else F32, n, D,
+                                         _stream()), "tanh_norm_chain")
+    return out if then is not None else None
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap tanh(x / cap)`` of fp32 numbers, in place."""
+    _need(x, "soft cap", torch.float32)
+    check(_lib.load().mm_soft_cap(x.data_ptr(), x.numel(), float(cap), _stream()), "soft_cap")
+    return x
+
+
+# ---- norms of queries and keys, rotation, cache write (csrc/attention_prep.cu) ----------------------------------------------------
+def qk_prep(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float,
+            rot: Optional[torch.Tensor], rot_dims: int, unit: bool, q_out: torch.Tensor, k_pages: Optional[torch.Tensor],
+            v_pages: Optional[torch.Tensor], slots: Optional[torch.Tensor], page_size: int, heads: int, kv_heads: int, key_dim: int,
+            value_dim: int) -> None:
+    """From rows [n, ld] (fp32, or the dtype of ``q_out``): with ``q_norm`` / ``k_norm`` (fp32, one number per row of the projection)
+    all q (all k) numbers of a token are divided by their common root mean square and weighed; the first ``rot_dims`` numbers of
+    every head are turned by ``rot`` [n, rot_dims/2, 2] (number i pairs with i + rot_dims/2); with ``unit`` every q and k head is
+    then divided by its root mean square.  q goes to ``q_out`` [n, heads * key_dim], k and v into their pages at ``slots``
+    (``k_pages`` None: the row holds q alone)."""
+    if rows.dtype not in (torch.float32, q_out.dtype) or not rows.is_cuda or rows.stride(1) != 1:
+        raise KernelError("qk prep: rows of fp32 or the activation dtype with unit column stride are needed")
+    n = rows.shape[0]
+    _need(q_out, "q_out")
+    if q_out.shape != (n, heads * key_dim):
+        raise KernelError("qk prep: q_out has another shape")
+    for w, what, count in ((q_norm, "q norm", heads * key_dim), (k_norm, "k norm", kv_heads * key_dim)):
+        if w is not None:
+            _need(w, what, torch.float32)
+            if w.numel() != count:
+                raise KernelError(f"qk prep: the {what} weight has one number per row of the projection")
+    if rot_dims:
+        _need(rot, "rotation table", torch.float32)
+        if rot.shape != (n, rot_dims // 2, 2):
+            raise KernelError("qk prep: rotation table of another shape")
+    ends = [q_off + heads * key_dim]
+    if k_pages is not None:
+        ends += [k_off + kv_heads * key_dim, v_off + kv_heads * value_dim]
+        _need(k_pages, "k_pages", q_out.dtype)
+        _need(v_pages, "v_pages", q_out.dtype)
+        _need(slots, "slots", torch.int32)
+        if k_pages.shape[1:] != (kv_heads, page_size, key_dim) or v_pages.shape[1:] != (kv_heads, page_size, value_dim):
+            raise KernelError("qk prep: page pool shape mismatch")
+    if max(ends) > rows.shape[1]:
+        raise KernelError("qk prep: columns outside the row")
+    check(_lib.load().mm_qk_prep(rows.data_ptr(), dtype_code(rows.dtype), rows.stride(0), int(q_off), int(k_off), int(v_off), _ptr(q_norm), _ptr(k_norm),
+                                 float(eps), _ptr(rot) if rot_dims else None, int(rot_dims), int(bool(unit)), q_out.data_ptr(), _ptr(k_pages),
+                                 _ptr(v_pages), dtype_code(q_out.dtype), _ptr(slots) if k_pages is not None else None, int(page_size), n,
+                                 int(heads), int(kv_heads), int(key_dim), int(value_dim), _stream()), "qk_prep")

@@ -77,6 +77,12 @@ class KVCacheSpec:
     head_dim: int = 0
     window: int = 0  # 0: every earlier token; W: the last W tokens (the current one included)
     arrays: Tuple[CacheArray, ...] = ()
+    chunk: int = 0   # C: the tokens of the query's own run of C, counted from position 0 (0: no runs)
+    keep: int = 0    # the first tokens of a sequence that are seen whatever the window or the run
+
+    def mask(self) -> Tuple[int, int, int]:
+        """(window, chunk, keep); an unlimited view is (0, 0, 0)."""
+        return (self.window, self.chunk, self.keep) if self.window or self.chunk else (0, 0, 0)
 
     def token_arrays(self) -> Tuple[CacheArray, ...]:
         if self.arrays:
@@ -176,6 +182,17 @@ class NormedRows:
 
 
 @dataclass
+class ElementwiseSink:
+    """Where a sublayer's last product adds its output itself, between norms that work number by number (``Norm.elementwise``): the
+    fp32 residual stream (in place) gets ``post(product)`` and, if ``then`` is given, the part returns ``then(residual)`` in the
+    activation dtype (or None).  Both norms are (weight, offset, alpha)."""
+
+    residual: torch.Tensor
+    post: Any
+    then: Any = None
+
+
+@dataclass
 class SplitBranch:
     """A sublayer's output still in pieces, for a block whose own launch puts them together:
     ``sum_c weights[t, c] rows[place[t, c]] + gate[t] other[t]``.  Without ``weights`` ``rows`` is [n, width] as it stands; without
@@ -243,6 +260,11 @@ class Norm(Part):
         prepare it in factored form (FactoredRows); None for any other norm."""
         return None
 
+    def elementwise(self) -> Optional[Tuple[torch.Tensor, torch.Tensor, float]]:
+        """(weight, offset, alpha), fp32, if the norm is ``weight * tanh(alpha * x) + offset``: it needs no other number of the row,
+        so that a product's epilogue can apply it; None for any other norm."""
+        return None
+
 
 class PositionEncoding(Part):
     def fused_rotary(self) -> Optional[Tuple[int, float]]:
@@ -270,6 +292,10 @@ class Mixer(Part):
         (ResidualSink).  Parts that do not override this are never given either."""
         return False
 
+    def fuses_elementwise(self, n_tokens: int) -> bool:
+        """True if, for a step of ``n_tokens``, ``forward`` takes a keyword ``sink`` (ElementwiseSink)."""
+        return False
+
 
 class FeedForward(Part):
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
@@ -278,6 +304,10 @@ class FeedForward(Part):
     def fuses(self, n_tokens: int) -> bool:
         """True if, for a step of ``n_tokens``, ``forward`` takes FactoredRows as ``x`` and a keyword ``sink``
         (ResidualSink).  Parts that do not override this are never given either."""
+        return False
+
+    def fuses_elementwise(self, n_tokens: int) -> bool:
+        """True if, for a step of ``n_tokens``, ``forward`` takes a keyword ``sink`` (ElementwiseSink)."""
         return False
 
 

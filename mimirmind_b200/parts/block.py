@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from ..registry import BLOCKS
-from .base import Block, FactoredRows, LayerCache, NativeDesc, NormedRows, ResidualSink, SplitBranch, StepContext
+from .base import Block, ElementwiseSink, FactoredRows, LayerCache, NativeDesc, NormedRows, ResidualSink, SplitBranch, StepContext
 
 
 @BLOCKS.register("pre_norm")
@@ -75,7 +75,8 @@ class SandwichNormBlock(Block):
     ``mixer_post_norm`` and ``ffn_post_norm``.
 
     The branch is normed, added into the fp32 residual stream and the sum normed for the next sublayer in one launch
-    where the two norms are grouped RMS norms of one shape; the last add of the layer does so for the first norm of
+    where the two norms are of one kind and shape (``same_shape``), and in the epilogue of the sublayer's last product where the norms
+    work number by number and the sublayer says it can (``fuses_elementwise``); the last add of the layer does so for the first norm of
     the block that follows and hands its rows over as ``NormedRows``.  The residual stream is complete when the block
     returns."""
 
@@ -94,7 +95,17 @@ class SandwichNormBlock(Block):
         return hasattr(self.mixer_norm, "same_shape")
 
     @staticmethod
-    def _add(post, residual: torch.Tensor, branch: torch.Tensor, then):
+    def _sink(part, post, then, residual: torch.Tensor, ctx: StepContext) -> Optional[ElementwiseSink]:
+        """The sublayer's sink, if its last product can do the post norm, the sum and the next norm itself."""
+        if ctx.plain_only or ctx.dump is not None or not part.fuses_elementwise(residual.shape[0]):
+            return None
+        p, t = post.elementwise(), then.elementwise() if then is not None else None
+        if p is None or (then is not None and t is None):
+            return None
+        return ElementwiseSink(residual, p, t)
+
+    @staticmethod
+    def _add(post, residual: torch.Tensor, branch, then):
         """residual += post(branch); returns then(residual) if ``then`` is given."""
         if hasattr(post, "add_normed") and (then is None or hasattr(then, "same_shape")):
             return post.add_normed(residual, branch, then)
@@ -110,19 +121,28 @@ class SandwichNormBlock(Block):
         dump = ctx.dump or (lambda stage, t: None)
         h = pending.x if isinstance(pending, NormedRows) else self.mixer_norm.forward(residual, pending)
         dump("attn_norm", h)
-        branch = self.mixer.forward(h, ctx, cache)
-        dump("attn_out", branch)
         hand_over = None
         if successor is not None and isinstance(successor, SandwichNormBlock) and successor.accepts_normed_rows() and not ctx.plain_only:
             hand_over = successor.mixer_norm
-        if self.has_ffn:
-            h = self._add(self.mixer_post, residual, branch, self.ffn_norm)
-            branch = self.feed_forward.forward(h, ctx)
-            dump("ffn_mlp", branch)
-            post = self.ffn_post
+        then = self.ffn_norm if self.has_ffn else hand_over
+        sink = self._sink(self.mixer, self.mixer_post, then, residual, ctx)
+        if sink is not None:
+            made = self.mixer.forward(h, ctx, cache, sink=sink)
         else:
-            post = self.mixer_post
-        made = self._add(post, residual, branch, hand_over)
+            branch = self.mixer.forward(h, ctx, cache)
+            dump("attn_out", branch)
+            made = self._add(self.mixer_post, residual, branch, then)
+        if self.has_ffn:
+            sink = self._sink(self.feed_forward, self.ffn_post, hand_over, residual, ctx)
+            if sink is not None:
+                made = self.feed_forward.forward(made, ctx, sink=sink)
+            else:
+                # a norm that works number by number also takes a branch in pieces and puts them together
+                ffn = self.feed_forward
+                split = self.ffn_post.elementwise() is not None and ctx.dump is None and hasattr(ffn, "splits_weighed") and ffn.splits_weighed()
+                branch = ffn.forward_split(made, ctx) if split else ffn.forward(made, ctx)
+                dump("ffn_mlp", branch)
+                made = self._add(self.ffn_post, residual, branch, hand_over)
         if ctx.dump is not None:
             dump("l_out", residual)
         return NormedRows(made) if made is not None else None

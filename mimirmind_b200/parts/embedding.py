@@ -84,7 +84,8 @@ class BigramEmbedding(Embedding):
 
 @HEADS.register("lm_head")
 class LMHead(Part):
-    """spec params: vocab, width, weight (full tensor name), tied_to (embedding tensor name or None)."""
+    """spec params: vocab, width, weight (full tensor name), tied_to (embedding tensor name or None), softcap (0: none; c: the
+    logits are bent into ``c tanh(logits / c)``)."""
 
     @classmethod
     def tensor_specs(cls, spec: PartSpec, prefix: str) -> List[TensorSpec]:
@@ -94,6 +95,7 @@ class LMHead(Part):
     def __init__(self, spec: PartSpec, weights: WeightView, rt: Runtime):
         super().__init__(spec, weights, rt)
         self.vocab = int(spec["vocab"])
+        self.softcap = float(spec.get("softcap", 0.0) or 0.0)
         if weights.has(spec["weight"]):
             self.weight = weights.get(spec["weight"]).contiguous()
         elif spec.get("tied_to") is not None:
@@ -102,7 +104,8 @@ class LMHead(Part):
             raise KeyError(f"tensor '{spec['weight']}' not in model")
 
     def native(self):
-        return NativeDesc("lm_head", {"vocab": self.vocab}, {"weight": self.weight}) if type(self) is LMHead else None
+        return NativeDesc("lm_head", {"vocab": self.vocab}, {"weight": self.weight}) if type(self) is LMHead and not self.softcap else None
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
-        return linear(x, self.weight, None, self.rt, out_dtype=torch.float32)
+        logits = linear(x, self.weight, None, self.rt, out_dtype=torch.float32)
+        return ops.soft_cap(logits, self.softcap) if self.softcap else logits

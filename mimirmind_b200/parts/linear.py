@@ -15,7 +15,7 @@ from typing import Optional
 import torch
 
 from ..kernels import ops
-from .base import Runtime
+from .base import ElementwiseSink, Runtime
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], rt: Runtime,
@@ -27,3 +27,11 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], 
         return matmul_bf16.matmul_nt(x, weight, bias, out_dtype)
     out = torch.empty((m, n), dtype=out_dtype, device=x.device)
     return ops.gemm_simt(x, weight, bias, out)
+
+
+def linear_into(x: torch.Tensor, weight: torch.Tensor, rt: Runtime, sink: Optional[ElementwiseSink]):
+    """A sublayer's last product: its rows, or with a sink (base.ElementwiseSink) its norm, the sum into the residual stream and the
+    next norm in the product's epilogue (the normed rows, or None where no norm follows)."""
+    if sink is None:
+        return linear(x, weight, None, rt)
+    return ops.gemv_bf16_tanh(x, weight, sink.residual, sink.post, sink.then)

@@ -13,8 +13,8 @@ import torch
 from ..config.spec import PartSpec, TensorSpec
 from ..kernels import ops
 from ..registry import FEED_FORWARDS
-from .base import FactoredRows, FeedForward, NativeDesc, ResidualSink, Runtime, StepContext, WeightView
-from .linear import linear
+from .base import ElementwiseSink, FactoredRows, FeedForward, NativeDesc, ResidualSink, Runtime, StepContext, WeightView
+from .linear import linear, linear_into
 
 
 @FEED_FORWARDS.register("swiglu")
@@ -144,22 +144,27 @@ class DenseMLP(FeedForward):
             self.b_up = weights.take(spec["up"] + sfx).contiguous()
             self.b_down = weights.take(spec["down"] + sfx).contiguous()
 
-    def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+    def fuses_elementwise(self, n_tokens: int) -> bool:
+        return self.b_down is None and ops.gemv_tanh_supported(self.rt, self.w_down, n_tokens)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, sink: Optional[ElementwiseSink] = None):
+        if sink is not None:
+            return linear_into(self._hidden(x, ctx), self.w_down, self.rt, sink)
+        return linear(self._hidden(x, ctx), self.w_down, self.b_down, self.rt)
+
+    def _hidden(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         if (x.dtype == torch.bfloat16 and self.w_up.dtype == torch.bfloat16 and self.rt.matmul != "simt" and not ctx.plain_only
                 and ops.small_batch_supported(x.shape[0], self.ff, self.hidden)):
             # a few tokens: bias and activation in the epilogue of the weight-streaming product
-            hidden = ops.gemv_bf16_act(x, self.w_up, self.b_up, self.activation)
-            return linear(hidden, self.w_down, self.b_down, self.rt)
+            return ops.gemv_bf16_act(x, self.w_up, self.b_up, self.activation)
         if (x.dtype == torch.bfloat16 and self.w_up.dtype == torch.bfloat16 and self.rt.matmul != "simt" and not ctx.plain_only
                 and x.shape[0] >= ops.TCGEN05_SWIGLU_MIN_ROWS and self.hidden >= FUSED_UP_MIN_HIDDEN
                 and ops.gemm_tcgen05_supported(x.shape[0], self.ff, self.hidden)):
             # prompt-sized and deep enough: the tcgen05 product with bias and activation as its epilogue (the hidden rows
             # never exist without their activation), as the gated feed-forward does with SwiGLU
-            hidden = ops.gemm_tcgen05_act(x, self.w_up, self.b_up, self.activation)
-            return linear(hidden, self.w_down, self.b_down, self.rt)
+            return ops.gemm_tcgen05_act(x, self.w_up, self.b_up, self.activation)
         hidden = linear(x, self.w_up, None, self.rt)
-        ops.bias_act(hidden, self.b_up, self.activation, hidden)
-        return linear(hidden, self.w_down, self.b_down, self.rt)
+        return ops.bias_act(hidden, self.b_up, self.activation, hidden)
 
 
 @FEED_FORWARDS.register("none")

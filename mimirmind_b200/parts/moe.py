@@ -6,7 +6,7 @@ are chosen and weighted by ``s / (sum of the chosen s + 1e-20)``.  Expert: ``W_d
 The output is the weighted sum of the chosen experts' outputs.
 
 Further options, each a parameter.  ``scoring`` ``sigmoid``: ``s = sigmoid(z)`` and the chosen experts are weighted by their
-``s`` as it is.  ``weight_on`` ``input``: the weight multiplies the expert's input, the output is ``sum_e expert_e(w_e h)``
+``s`` as it is, or with ``renorm`` by ``s`` over the chosen ones' sum.  ``weight_scale`` multiplies the weights.  ``weight_on`` ``input``: the weight multiplies the expert's input, the output is ``sum_e expert_e(w_e h)``
 (both of an expert's first products are linear, so the weight is applied to their results in fp32).  ``activation``
 ``clamped`` with ``limit``: ``g = min(W_gate h, limit)``, ``u = clamp(W_up h, -limit, limit)``, ``y = g sigmoid(1.702 g) (u + 1)``.
 ``shared``: the PartSpec of a feed-forward that every token goes through beside its routed experts; the two results add up.
@@ -45,7 +45,7 @@ def ctx_plain(ctx) -> bool:
 class RoutedExperts(FeedForward):
     """spec params: hidden, ff, experts, top, groups, keep, router (tensor name), expert (a name pattern with ``{}`` for
     the expert's number, e.g. ``mlp.e{}``; its matrices are ``.gate`` (if gated), ``.up``, ``.down``), scoring (``softmax`` or
-    ``sigmoid``), weight_on (``output`` or ``input``), gated (default True), activation (gated: ``silu``, ``clamped`` or ``gelu_tanh``;
+    ``sigmoid``), renorm (default: as the scoring has it), weight_scale (default 1), weight_on (``output`` or ``input``), gated (default True), activation (gated: ``silu``, ``clamped`` or ``gelu_tanh``;
     else one of a plain feed-forward's), limit, correction (tensor name or None), group_score (``max`` or ``top2_sum``), shared
     (PartSpec or None), shared_gate (tensor name or None)."""
 
@@ -75,6 +75,8 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed experts: the experts split into equal runs, 0 < keep <= runs, and top fits into the kept runs")
         self.scoring, self.weight_on = spec.get("scoring", "softmax"), spec.get("weight_on", "output")
         self.activation, self.limit = spec.get("activation", "silu"), float(spec.get("limit", 0.0) or 0.0)
+        self.renorm = spec.get("renorm")
+        self.weight_scale = float(spec.get("weight_scale", 1.0))
         self.gated, self.group_score = bool(spec.get("gated", True)), spec.get("group_score", "max")
         known = ops.GLU_ACTIVATIONS if self.gated else ops.ACTIVATIONS
         if (self.scoring not in ops.ROUTER_SCORINGS or self.weight_on not in ("output", "input") or self.activation not in known
@@ -118,6 +120,10 @@ class RoutedExperts(FeedForward):
         y, gate = self._combined(x, ctx)
         return y if self.shared is None else ops.scaled_sum2(y, self.shared.forward(x, ctx), 1.0, 1.0, gate)
 
+    def splits_weighed(self) -> bool:
+        """True if the result in pieces (``forward_split``) is the chosen rows with their weights and nothing else."""
+        return self.shared is None and self.weight_on == "output"
+
     def forward_split(self, x: torch.Tensor, ctx: StepContext) -> SplitBranch:
         """The result in pieces: every token's chosen rows with their weights, and the shared expert's with its gate."""
         y, wts, place, gate = self._routed(x, ctx)
@@ -134,7 +140,7 @@ class RoutedExperts(FeedForward):
         shared expert's gate per token or None)."""
         n = x.shape[0]
         chosen = ops.moe_router(x, self.w_router, self.top, self.groups, self.keep, scoring=self.scoring, correction=self.correction,
-                                group_score=self.group_score, gate=self.shared_gated)
+                                group_score=self.group_score, gate=self.shared_gated, renorm=self.renorm, scale=self.weight_scale)
         idx, wts, gate = chosen if self.shared_gated else chosen + (None,)
         n_rows = n * self.top
         on_input = self.weight_on == "input"

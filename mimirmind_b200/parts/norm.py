@@ -14,7 +14,7 @@ import torch
 from ..config.spec import PartSpec, TensorSpec
 from ..kernels import ops
 from ..registry import NORMS
-from .base import NativeDesc, Norm, Runtime, WeightView
+from .base import NativeDesc, Norm, Runtime, SplitBranch, WeightView
 
 
 @NORMS.register("rmsnorm")
@@ -110,6 +110,60 @@ class GroupRMSNorm(Norm):
             return then.forward(residual, None)
         out = torch.empty((residual.shape[0], self.width), dtype=self.rt.dtype, device=residual.device)
         return ops.group_norm_chain(residual, branch, self.weight, then.weight, self.groups, self.eps, out)
+
+
+@NORMS.register("tanh_norm")
+class TanhNorm(Norm):
+    """A norm without statistics: ``w tanh(alpha x) + b`` with one slope ``alpha`` for the tensor and a weight and an offset per channel.
+    Every number is normed on its own, so the norm of a branch, the sum into the residual stream and the next such norm are one
+    elementwise launch, or the epilogue of the product that makes the branch.
+
+    spec params: width, weight, offset, alpha (tensor names under the prefix)."""
+
+    @classmethod
+    def tensor_specs(cls, spec: PartSpec, prefix: str) -> List[TensorSpec]:
+        d = spec["width"]
+        return [TensorSpec(prefix + spec["weight"], (d,), role="norm"), TensorSpec(prefix + spec["offset"], (d,), role="bias"),
+                TensorSpec(prefix + spec["alpha"], (), role="norm")]
+
+    def __init__(self, spec: PartSpec, weights: WeightView, rt: Runtime):
+        super().__init__(spec, weights, rt)
+        self.width = int(spec["width"])
+        self.weight = weights.get(spec["weight"]).float().contiguous()
+        self.offset = weights.get(spec["offset"]).float().contiguous()
+        self.alpha = float(weights.get(spec["alpha"]).float().item())       # read once at load: kernels take it by value
+
+    def elementwise(self):
+        return (self.weight, self.offset, self.alpha)
+
+    def same_shape(self, other) -> bool:
+        """True if ``other`` is a norm that one launch can chain with this one."""
+        return isinstance(other, TanhNorm) and other.width == self.width
+
+    def forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None,
+                n_rows: Optional[int] = None) -> torch.Tensor:
+        if rows is not None:
+            if n_rows is not None and rows.numel() != n_rows:
+                rows = rows[:n_rows]
+            if delta is not None:
+                ops.add_residual(residual, delta)
+        n = residual.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.width), dtype=self.rt.dtype, device=residual.device)
+        return ops.tanh_norm_chain(residual, delta if rows is None else None, None, self.elementwise(), out, rows=rows)
+
+    def add_normed(self, residual: torch.Tensor, branch, then: Optional["TanhNorm"] = None) -> Optional[torch.Tensor]:
+        """``residual += norm(branch)`` with this norm; with ``then`` also returns ``then(residual)`` from the same launch.  The branch
+        is a tensor or a SplitBranch of weighed rows."""
+        wts = place = None
+        if isinstance(branch, SplitBranch):
+            if branch.other is not None or branch.weights is None:
+                raise ValueError("tanh norm: only weighed rows are taken in pieces")
+            branch, wts, place = branch.rows, branch.weights, branch.place
+        if then is not None and not self.same_shape(then):
+            ops.tanh_norm_chain(residual, branch, self.elementwise(), None, wts=wts, place=place)
+            return then.forward(residual, None)
+        out = torch.empty((residual.shape[0], self.width), dtype=self.rt.dtype, device=residual.device) if then is not None else None
+        return ops.tanh_norm_chain(residual, branch, self.elementwise(), then.elementwise() if then is not None else None, out, wts=wts, place=place)
 
 
 @NORMS.register("none")

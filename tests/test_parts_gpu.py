@@ -639,7 +639,7 @@ def test_a_layer_named_twice_and_an_entry_that_reads_another_entrys_cache(sizes,
             assert np.array_equal(got, first), cuts                     # 32-bit: the same bits however the tokens are cut
     runner.check_errors()
 
-    # an entry may not look further back than the entry whose cache it reads keeps
-    bad = ModelSpec("ScheduledBad", d, V, 512, spec.embedding, layers, (ScheduleEntry(1), ScheduleEntry(0, 0)), spec.final_norm, spec.head)
-    with pytest.raises(ValueError, match="keeps only"):
-        Model(bad, {k: v.clone() for k, v in tensors.items()}, rt_)
+    # an entry that looks further back than the entry whose cache it reads makes that cache keep more
+    wide = ModelSpec("ScheduledWide", d, V, 512, spec.embedding, layers, (ScheduleEntry(1), ScheduleEntry(0, 0)), spec.final_norm, spec.head)
+    (group,) = Model(wide, {k: v.clone() for k, v in tensors.items()}, rt_).cache_groups()
+    assert group.masks == ((0, 0, 0),)
