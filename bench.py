@@ -166,7 +166,7 @@ def run_workload(name: str, layers: int) -> int:
     return 0 if verified else 1
 
 
-# ---- another design beside the closest existing one, at equal size (--compare bigerax | domelix | segorax | tupunex | zubarax) ---------------------------------------
+# ---- another design beside the closest existing one, at equal size (--compare bigerax | domelix | nefelorn | nefelorn_experts | segorax | tupunex | zubarax) ---------------------------------------
 # Layer sizes that resemble a real model's; both models get the same width, heads, key size, window, layer count and
 # vocabulary, and feed-forwards of equal parameter count (two matrices of ff against three of 2/3 ff).
 COMPARE_SIZES = {
@@ -258,6 +258,30 @@ def tupunex_latent_config(z):
     return out
 
 
+def nefelorn_config(z, experts=False):
+    """The four kinds of layers in turn: a window beside 4 kept tokens, runs of the window's length, the same with the keys and values of
+    the layer before, a window again; every layer with a dense feed-forward, or (``experts``) with Domelix's routed experts (16 of
+    three matrices, 4 chosen)."""
+    d, expert_ff = z["width"], -(-(2 * z["ff"] // 12) // 64) * 64
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": 16, "top": 4, "scale": 2.0}} if experts else {"kind": "dense", "ff": z["ff"]}
+    size = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5}
+    far = dict(size, mask={"size": z["window"]},
+               rot={"base": 500000.0, "dims": z["dim"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    near = {"type": "attention_2", "mlp": mlp,
+            "mixer": dict(size, mask={"size": z["window"], "keep_first": 4}, rot={"base": 500000.0, "dims": z["dim"] // 2})}
+    layers = [near if i % 4 in (0, 3) else {"type": "attention", "mlp": mlp, "mixer": far if i % 4 == 1 else dict(far, kv_from=i - 1)}
+              for i in range(z["layers"])]
+    return {"architecture": "Nefelorn", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "logit_softcap": 30.0,
+            "layers": layers}
+
+
+def bigerax_attention_config(z):
+    """Bigerax with attention and a feed-forward in every layer."""
+    out = bigerax_config(dict(z, layers=4))
+    out["layers"] = [out["layers"][0]] * z["layers"]
+    return out
+
+
 def qwen2_config(z, context):
     inter = -(-(2 * z["ff"] // 3) // 64) * 64
     return dict(architectures=["Qwen2ForCausalLM"], model_type="qwen2", num_hidden_layers=z["layers"], hidden_size=z["width"],
@@ -269,7 +293,8 @@ def qwen2_config(z, context):
 def run_compare(args) -> int:
     """Prefill and decode throughput of one design beside the closest other one at equal size (random weights, bfloat16):
     Bigerax beside the Qwen2 decoder, Domelix beside Bigerax, Tupunex beside the Qwen2 decoder, Zubarax beside Domelix,
-    Segorax beside Tupunex with latent attention in every layer; one prompt in one step (median of five), and the captured
+    Segorax beside Tupunex with latent attention in every layer, Nefelorn with dense feed-forwards beside Bigerax with attention in
+    every layer, and with experts beside Domelix; one prompt in one step (median of five), and the captured
     decode step at the given batch over prompts of that length."""
     import numpy as np
     import torch
@@ -286,10 +311,12 @@ def run_compare(args) -> int:
     steps, warmup, batch = max(1, min(args.steps, 128)), max(3, args.warmup), max(1, args.batch)
     context = -(-(prompt_len + SETTLE_STEPS + warmup + steps + 1) // 1024) * 1024
     first, second = {"bigerax": ("bigerax", "qwen2"), "domelix": ("domelix", "bigerax"), "tupunex": ("tupunex", "qwen2"),
-                     "zubarax": ("zubarax", "domelix"), "segorax": ("segorax", "tupunex_latent")}[args.compare]
+                     "zubarax": ("zubarax", "domelix"), "segorax": ("segorax", "tupunex_latent"), "nefelorn": ("nefelorn", "bigerax_attention"),
+                     "nefelorn_experts": ("nefelorn_experts", "domelix")}[args.compare]
     configs = {"bigerax": lambda z: bigerax_config(z), "qwen2": lambda z: qwen2_config(z, context), "domelix": lambda z: domelix_config(z),
                "tupunex": lambda z: tupunex_config(z), "zubarax": lambda z: zubarax_config(z), "segorax": lambda z: segorax_config(z),
-               "tupunex_latent": lambda z: tupunex_latent_config(z)}
+               "tupunex_latent": lambda z: tupunex_latent_config(z), "nefelorn": lambda z: nefelorn_config(z),
+               "nefelorn_experts": lambda z: nefelorn_config(z, experts=True), "bigerax_attention": lambda z: bigerax_attention_config(z)}
     out = {"compare": first, "beside": second, "dtype": "bf16", "data": "synthetic", "prompt_len": prompt_len, "batch": batch,
            "steps": steps, "warmup": warmup, "sizes": {}}
     sizes = [args.size] if args.size else sorted(COMPARE_SIZES)
@@ -409,9 +436,9 @@ def main() -> int:
                     help="with --only decode or prefill: prompts of this many tokens instead of 2,048 (the context grows with them)")
     ap.add_argument("--opt", action="append", default=[], metavar="NAME=VALUE",
                     help="set a tunable of the library's dispatch (csrc/exec/exec.h, Options) for this run, e.g. cluster_max_wanted=64")
-    ap.add_argument("--compare", default="", choices=["", "bigerax", "domelix", "segorax", "tupunex", "zubarax"],
+    ap.add_argument("--compare", default="", choices=["", "bigerax", "domelix", "nefelorn", "nefelorn_experts", "segorax", "tupunex", "zubarax"],
                     help="instead of the default run: prefill and decode throughput of that design beside the closest other one (bigerax "
-                         "beside the Qwen2 decoder, domelix beside bigerax, tupunex beside the Qwen2 decoder, zubarax beside domelix, segorax beside tupunex with latent attention in every layer) at equal size, at layer sizes that resemble a real model's (random weights; --size, --layers, --batch, --prompt-len, --steps)")
+                         "beside the Qwen2 decoder, domelix beside bigerax, tupunex beside the Qwen2 decoder, zubarax beside domelix, segorax beside tupunex with latent attention in every layer, nefelorn beside bigerax with attention in every layer, nefelorn_experts beside domelix) at equal size, at layer sizes that resemble a real model's (random weights; --size, --layers, --batch, --prompt-len, --steps)")
     ap.add_argument("--size", default="", choices=[""] + sorted(COMPARE_SIZES), help="with --compare: one size only")
     args = ap.parse_args()
 

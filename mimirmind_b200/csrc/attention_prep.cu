@@ -67,58 +67,93 @@ __device__ __forceinline__ float span_inverse_rms(const TI* p, int count, float 
     return 1.0f / sqrtf(block_sum(ss, scratch) / (float)count + eps);
 }
 
+// Two sums over the block at once (a fixed order: lanes, then warps)
+__device__ __forceinline__ float2 block_sum2(float x, float y, float2* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+    x = warp_sum(x);
+    y = warp_sum(y);
+    if (lane == 0) scratch[warp] = make_float2(x, y);
+    __syncthreads();
+    const float2 t = lane < nwarps ? scratch[lane] : make_float2(0.0f, 0.0f);
+    return make_float2(warp_sum(t.x), warp_sum(t.y));
+}
+
 // Head sizes of which every piece is a multiple of four numbers: a head is dk / 8 units of eight numbers (four pairs, or eight
-// numbers that do not turn), one lane each, `lanes` (a power of two) lanes per head.
-template <typename TI, typename T>
-__global__ void __launch_bounds__(PREP_THREADS) qk_prep_vec_kernel(const TI* __restrict__ rows, T* __restrict__ q_out, T* __restrict__ k_pages,
-                                                                   T* __restrict__ v_pages, const PrepArgs a, int lanes) {
-    __shared__ float scratch[32];
+// numbers that do not turn), one lane each, `lanes` (a power of two) lanes per head.  ONE: the block has lanes for every head, so
+// that a row is read once and the sums of the span norms come from the registers it stands in.
+template <typename TI, typename T, bool ONE>
+__global__ void __launch_bounds__(ONE ? 1024 : PREP_THREADS) qk_prep_vec_kernel(const TI* __restrict__ rows, T* __restrict__ q_out, T* __restrict__ k_pages,
+                                                                                T* __restrict__ v_pages, const PrepArgs a, int lanes) {
+    __shared__ float2 scratch[32];
     const int t = blockIdx.x, H = a.H, G = k_pages != nullptr ? a.G : 0, dk = a.dk, dv = a.dv, half = a.rot_dims / 2;
     const TI* row = rows + (size_t)t * a.ld;
-    float rq = 1.0f, rk = 1.0f;
-    if (a.wq != nullptr) rq = span_inverse_rms<TI, true>(row + a.q_off, H * dk, a.eps, scratch);
-    if (a.wk != nullptr && G > 0) rk = span_inverse_rms<TI, true>(row + a.k_off, G * dk, a.eps, scratch);
     const long long slot = G > 0 ? (long long)a.slots[t] : -1;
     const long long page = slot >= 0 ? slot / a.page_size : -1;
     const int place = slot >= 0 ? (int)(slot - page * a.page_size) : 0;
     const int lane = threadIdx.x & (lanes - 1), groups = blockDim.x / lanes, units = dk / 8;
+    const bool spans = a.wq != nullptr || (a.wk != nullptr && G > 0), turns = lane * 4 < half;
+    const int at0 = turns ? lane * 4 : a.rot_dims + (lane - half / 4) * 8, at1 = turns ? at0 + half : at0 + 4;
+    float rq = 1.0f, rk = 1.0f;
+    if (!ONE && spans) {
+        float* one = reinterpret_cast<float*>(scratch);
+        if (a.wq != nullptr) rq = span_inverse_rms<TI, true>(row + a.q_off, H * dk, a.eps, one);
+        if (a.wk != nullptr && G > 0) rk = span_inverse_rms<TI, true>(row + a.k_off, G * dk, a.eps, one);
+    }
+    if (page >= 0) {
+        for (int i = threadIdx.x * 4; i < G * dv; i += blockDim.x * 4) {
+            const int g = i / dv, e = i - g * dv;
+            float v[4];
+            prep_load4<TI>(row + a.v_off + i, v);
+            prep_store4<T>(v_pages + (((size_t)page * G + g) * a.page_size + place) * dv + e, v);
+        }
+    }
     for (int h0 = 0; h0 < H + G; h0 += groups) {               // every thread takes every turn: the lanes of a head add up
         const int head = h0 + threadIdx.x / lanes;
         const bool live = head < H + G && lane < units, is_q = head < H;
-        float x[8];
-        int at0 = 0, at1 = 0;
-        float ss = 0.0f;
+        const int off = is_q ? head * dk : (head - H) * dk;
+        const float* w = is_q ? a.wq : a.wk;
+        float x[8], wv[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = wv[e] = 0.0f;
         if (live) {
-            const int off = is_q ? head * dk : (head - H) * dk;
             const TI* p = row + (is_q ? a.q_off : a.k_off) + off;
-            const bool turns = lane * 4 < half;
-            at0 = turns ? lane * 4 : a.rot_dims + (lane - half / 4) * 8;
-            at1 = turns ? at0 + half : at0 + 4;
             prep_load4<TI>(p + at0, x);
             prep_load4<TI>(p + at1, x + 4);
-            const float* w = is_q ? a.wq : a.wk;
             if (w != nullptr) {
-                float wv[8];
                 prep_load4<float>(w + off + at0, wv);
                 prep_load4<float>(w + off + at1, wv + 4);
+            }
+        }
+        if (ONE && spans) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
+            const float2 s = block_sum2(is_q ? ss : 0.0f, is_q ? 0.0f : ss, scratch);
+            rq = 1.0f / sqrtf(s.x / (float)(H * dk) + a.eps);
+            rk = 1.0f / sqrtf(s.y / (float)(a.G * dk) + a.eps);
+        }
+        if (live) {
+            if (w != nullptr) {
                 const float r = is_q ? rq : rk;
 #pragma unroll
                 for (int e = 0; e < 8; ++e) x[e] = x[e] * r * wv[e];
             }
             if (turns) {
-                const float2* cs = a.rot + (size_t)t * half + at0;
+                const float4* cs = reinterpret_cast<const float4*>(a.rot + (size_t)t * half + at0);
+                const float4 c01 = cs[0], c23 = cs[1];
+                const float c[4] = {c01.x, c01.z, c23.x, c23.z}, sn[4] = {c01.y, c01.w, c23.y, c23.w};
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float2 c = cs[e];
                     const float u = x[e], v = x[4 + e];
-                    x[e] = u * c.x - v * c.y;
-                    x[4 + e] = v * c.x + u * c.y;
+                    x[e] = u * c[e] - v * sn[e];
+                    x[4 + e] = v * c[e] + u * sn[e];
                 }
             }
-#pragma unroll
-            for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
         }
         if (a.unit) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
             for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
             const float r = 1.0f / sqrtf(ss / (float)dk + a.eps);
 #pragma unroll
@@ -130,13 +165,6 @@ __global__ void __launch_bounds__(PREP_THREADS) qk_prep_vec_kernel(const TI* __r
             prep_store4<T>(dst + at0, x);
             prep_store4<T>(dst + at1, x + 4);
         }
-    }
-    if (page < 0) return;
-    for (int i = threadIdx.x * 4; i < G * dv; i += blockDim.x * 4) {
-        const int g = i / dv, e = i - g * dv;
-        float v[4];
-        prep_load4<TI>(row + a.v_off + i, v);
-        prep_store4<T>(v_pages + (((size_t)page * G + g) * a.page_size + place) * dv + e, v);
     }
 }
 
@@ -193,9 +221,11 @@ static void prep_launch(const void* rows, void* q_out, void* k_pages, void* v_pa
     if (vec) {
         int lanes = 1;
         while (lanes < a.dk / 8) lanes *= 2;
-        int threads = PREP_THREADS;
-        while (threads > 64 && (threads / 2) / lanes >= a.H + (k_pages ? a.G : 0)) threads /= 2;
-        mm_launch(qk_prep_vec_kernel<TI, T>, dim3(n), dim3(threads), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a, lanes);
+        const int all = ((a.H + (k_pages ? a.G : 0)) * lanes + 31) / 32 * 32;
+        if (all <= 1024)
+            mm_launch(qk_prep_vec_kernel<TI, T, true>, dim3(n), dim3(all), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a, lanes);
+        else
+            mm_launch(qk_prep_vec_kernel<TI, T, false>, dim3(n), dim3(PREP_THREADS), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a, lanes);
     } else {
         mm_launch(qk_prep_kernel<TI, T>, dim3(n), dim3(PREP_THREADS), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a);
     }
@@ -215,7 +245,7 @@ MM_EXPORT int mm_qk_prep(const void* rows, int rows_dtype, int ld, int q_off, in
     a.rot = (const float2*)rot; a.rot_dims = rot_dims; a.unit = unit;
     a.slots = (const int32_t*)slots; a.page_size = page_size; a.H = H; a.G = G; a.dk = dk; a.dv = dv;
     const bool vec = dk % 8 == 0 && dk <= 256 && rot_dims % 8 == 0 && dv % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
-                     (((uintptr_t)rows | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)wq | (uintptr_t)wk) & 15) == 0;
+                     (((uintptr_t)rows | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)wq | (uintptr_t)wk | (uintptr_t)rot) & 15) == 0;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
     if (rows_dtype == MM_F32 && dtype == MM_F32) prep_launch<float, float>(rows, q_out, k_pages, v_pages, a, n_tokens, vec, s);

@@ -177,7 +177,7 @@ def router_choice(h, w_router, top, scale):
 
 
 def experts_feed_forward(h, w, p, f):
-    idx, wts = router_choice(h, w[p + "router"], f["router"]["top"], f["router"]["scale"])
+    idx, wts = router_choice(h, w[p + "router"], f["router"]["top"], f["router"].get("scale", 1.0))
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e, s in zip(idx[t], wts[t]):
