@@ -48,21 +48,12 @@ __device__ __forceinline__ void prep_store4<__nv_bfloat16>(__nv_bfloat16* p, con
 }
 
 // 1 / root mean square of `count` consecutive numbers, by the whole block
-template <typename TI, bool VEC>
+template <typename TI>
 __device__ __forceinline__ float span_inverse_rms(const TI* p, int count, float eps, float* scratch) {
     float ss = 0.0f;
-    if constexpr (VEC) {
-        for (int i = threadIdx.x * 4; i < count; i += blockDim.x * 4) {
-            float v[4];
-            prep_load4<TI>(p + i, v);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) ss = fmaf(v[e], v[e], ss);
-        }
-    } else {
-        for (int i = threadIdx.x; i < count; i += blockDim.x) {
-            const float x = to_f32<TI>(p[i]);
-            ss = fmaf(x, x, ss);
-        }
+    for (int i = threadIdx.x; i < count; i += blockDim.x) {
+        const float x = to_f32<TI>(p[i]);
+        ss = fmaf(x, x, ss);
     }
     return 1.0f / sqrtf(block_sum(ss, scratch) / (float)count + eps);
 }
@@ -79,26 +70,42 @@ __device__ __forceinline__ float2 block_sum2(float x, float y, float2* scratch) 
 }
 
 // Head sizes of which every piece is a multiple of four numbers: a head is dk / 8 units of eight numbers (four pairs, or eight
-// numbers that do not turn), one lane each, `lanes` (a power of two) lanes per head.  ONE: the block has lanes for every head, so
-// that a row is read once and the sums of the span norms come from the registers it stands in.
-template <typename TI, typename T, bool ONE>
-__global__ void __launch_bounds__(ONE ? 1024 : PREP_THREADS) qk_prep_vec_kernel(const TI* __restrict__ rows, T* __restrict__ q_out, T* __restrict__ k_pages,
-                                                                                T* __restrict__ v_pages, const PrepArgs a, int lanes) {
+// numbers that do not turn), one lane each, `lanes` (a power of two) lanes per head, TURNS heads per group of lanes (a compile-time
+// number, so that all of a row's loads are under way before the first is used, and the sums of the span norms come from the
+// registers the row stands in).
+template <typename TI, typename T, int TURNS>
+__global__ void __launch_bounds__(TURNS == 1 ? 1024 : PREP_THREADS) qk_prep_vec_kernel(const TI* __restrict__ rows, T* __restrict__ q_out,
+                                                                                       T* __restrict__ k_pages, T* __restrict__ v_pages, const PrepArgs a,
+                                                                                       int lanes) {
     __shared__ float2 scratch[32];
     const int t = blockIdx.x, H = a.H, G = k_pages != nullptr ? a.G : 0, dk = a.dk, dv = a.dv, half = a.rot_dims / 2;
     const TI* row = rows + (size_t)t * a.ld;
+    const int lane = threadIdx.x & (lanes - 1), groups = blockDim.x / lanes, head0 = threadIdx.x / lanes;
+    const bool spans = a.wq != nullptr || (a.wk != nullptr && G > 0), turns = lane * 4 < half, unit_lane = lane < dk / 8;
+    const int at0 = turns ? lane * 4 : a.rot_dims + (lane - half / 4) * 8, at1 = turns ? at0 + half : at0 + 4;
+    float x[TURNS][8];
+    float sq = 0.0f, sk = 0.0f;
+#pragma unroll
+    for (int u = 0; u < TURNS; ++u) {
+        const int head = head0 + u * groups;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[u][e] = 0.0f;
+        if (unit_lane && head < H + G) {
+            const TI* p = row + (head < H ? a.q_off + head * dk : a.k_off + (head - H) * dk);
+            prep_load4<TI>(p + at0, x[u]);
+            prep_load4<TI>(p + at1, x[u] + 4);
+        }
+    }
+    float cs[4], sn[4];
+    if (turns) {
+        const float4* c = reinterpret_cast<const float4*>(a.rot + (size_t)t * half + at0);
+        const float4 c01 = c[0], c23 = c[1];
+        cs[0] = c01.x; sn[0] = c01.y; cs[1] = c01.z; sn[1] = c01.w;
+        cs[2] = c23.x; sn[2] = c23.y; cs[3] = c23.z; sn[3] = c23.w;
+    }
     const long long slot = G > 0 ? (long long)a.slots[t] : -1;
     const long long page = slot >= 0 ? slot / a.page_size : -1;
     const int place = slot >= 0 ? (int)(slot - page * a.page_size) : 0;
-    const int lane = threadIdx.x & (lanes - 1), groups = blockDim.x / lanes, units = dk / 8;
-    const bool spans = a.wq != nullptr || (a.wk != nullptr && G > 0), turns = lane * 4 < half;
-    const int at0 = turns ? lane * 4 : a.rot_dims + (lane - half / 4) * 8, at1 = turns ? at0 + half : at0 + 4;
-    float rq = 1.0f, rk = 1.0f;
-    if (!ONE && spans) {
-        float* one = reinterpret_cast<float*>(scratch);
-        if (a.wq != nullptr) rq = span_inverse_rms<TI, true>(row + a.q_off, H * dk, a.eps, one);
-        if (a.wk != nullptr && G > 0) rk = span_inverse_rms<TI, true>(row + a.k_off, G * dk, a.eps, one);
-    }
     if (page >= 0) {
         for (int i = threadIdx.x * 4; i < G * dv; i += blockDim.x * 4) {
             const int g = i / dv, e = i - g * dv;
@@ -107,63 +114,58 @@ __global__ void __launch_bounds__(ONE ? 1024 : PREP_THREADS) qk_prep_vec_kernel(
             prep_store4<T>(v_pages + (((size_t)page * G + g) * a.page_size + place) * dv + e, v);
         }
     }
-    for (int h0 = 0; h0 < H + G; h0 += groups) {               // every thread takes every turn: the lanes of a head add up
-        const int head = h0 + threadIdx.x / lanes;
-        const bool live = head < H + G && lane < units, is_q = head < H;
-        const int off = is_q ? head * dk : (head - H) * dk;
-        const float* w = is_q ? a.wq : a.wk;
-        float x[8], wv[8];
+    float rq = 1.0f, rk = 1.0f;
+    if (spans) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = wv[e] = 0.0f;
-        if (live) {
-            const TI* p = row + (is_q ? a.q_off : a.k_off) + off;
-            prep_load4<TI>(p + at0, x);
-            prep_load4<TI>(p + at1, x + 4);
-            if (w != nullptr) {
-                prep_load4<float>(w + off + at0, wv);
-                prep_load4<float>(w + off + at1, wv + 4);
-            }
-        }
-        if (ONE && spans) {
+        for (int u = 0; u < TURNS; ++u) {
             float ss = 0.0f;
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
-            const float2 s = block_sum2(is_q ? ss : 0.0f, is_q ? 0.0f : ss, scratch);
-            rq = 1.0f / sqrtf(s.x / (float)(H * dk) + a.eps);
-            rk = 1.0f / sqrtf(s.y / (float)(a.G * dk) + a.eps);
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[u][e], x[u][e], ss);
+            if (head0 + u * groups < H) sq += ss;
+            else sk += ss;
         }
+        const float2 s = block_sum2(sq, sk, scratch);
+        rq = 1.0f / sqrtf(s.x / (float)(H * dk) + a.eps);
+        rk = 1.0f / sqrtf(s.y / (float)(a.G * dk) + a.eps);
+    }
+#pragma unroll
+    for (int u = 0; u < TURNS; ++u) {                          // every thread takes every turn: the lanes of a head add up
+        const int head = head0 + u * groups;
+        const bool live = unit_lane && head < H + G, is_q = head < H;
         if (live) {
+            const float* w = is_q ? a.wq : a.wk;
             if (w != nullptr) {
+                const int off = is_q ? head * dk : (head - H) * dk;
+                float wv[8];
+                prep_load4<float>(w + off + at0, wv);
+                prep_load4<float>(w + off + at1, wv + 4);
                 const float r = is_q ? rq : rk;
 #pragma unroll
-                for (int e = 0; e < 8; ++e) x[e] = x[e] * r * wv[e];
+                for (int e = 0; e < 8; ++e) x[u][e] = x[u][e] * r * wv[e];
             }
             if (turns) {
-                const float4* cs = reinterpret_cast<const float4*>(a.rot + (size_t)t * half + at0);
-                const float4 c01 = cs[0], c23 = cs[1];
-                const float c[4] = {c01.x, c01.z, c23.x, c23.z}, sn[4] = {c01.y, c01.w, c23.y, c23.w};
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float u = x[e], v = x[4 + e];
-                    x[e] = u * c[e] - v * sn[e];
-                    x[4 + e] = v * c[e] + u * sn[e];
+                    const float p = x[u][e], v = x[u][4 + e];
+                    x[u][e] = p * cs[e] - v * sn[e];
+                    x[u][4 + e] = v * cs[e] + p * sn[e];
                 }
             }
         }
         if (a.unit) {
             float ss = 0.0f;
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[u][e], x[u][e], ss);
             for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
             const float r = 1.0f / sqrtf(ss / (float)dk + a.eps);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] *= r;
+            for (int e = 0; e < 8; ++e) x[u][e] *= r;
         }
         if (!live) continue;
         T* dst = is_q ? q_out + ((size_t)t * H + head) * dk : (page >= 0 ? k_pages + (((size_t)page * G + (head - H)) * a.page_size + place) * dk : nullptr);
         if (dst != nullptr) {
-            prep_store4<T>(dst + at0, x);
-            prep_store4<T>(dst + at1, x + 4);
+            prep_store4<T>(dst + at0, x[u]);
+            prep_store4<T>(dst + at1, x[u] + 4);
         }
     }
 }
@@ -176,8 +178,8 @@ __global__ void __launch_bounds__(PREP_THREADS) qk_prep_kernel(const TI* __restr
     const int t = blockIdx.x, H = a.H, G = k_pages != nullptr ? a.G : 0, dk = a.dk, dv = a.dv, half = a.rot_dims / 2;
     const TI* row = rows + (size_t)t * a.ld;
     float rq = 1.0f, rk = 1.0f;
-    if (a.wq != nullptr) rq = span_inverse_rms<TI, false>(row + a.q_off, H * dk, a.eps, scratch);
-    if (a.wk != nullptr && G > 0) rk = span_inverse_rms<TI, false>(row + a.k_off, G * dk, a.eps, scratch);
+    if (a.wq != nullptr) rq = span_inverse_rms<TI>(row + a.q_off, H * dk, a.eps, scratch);
+    if (a.wk != nullptr && G > 0) rk = span_inverse_rms<TI>(row + a.k_off, G * dk, a.eps, scratch);
     const long long slot = G > 0 ? (long long)a.slots[t] : -1;
     const long long page = slot >= 0 ? slot / a.page_size : -1;
     const int place = slot >= 0 ? (int)(slot - page * a.page_size) : 0;
@@ -218,17 +220,22 @@ __global__ void __launch_bounds__(PREP_THREADS) qk_prep_kernel(const TI* __restr
 
 template <typename TI, typename T>
 static void prep_launch(const void* rows, void* q_out, void* k_pages, void* v_pages, const PrepArgs& a, int n, bool vec, cudaStream_t s) {
-    if (vec) {
-        int lanes = 1;
-        while (lanes < a.dk / 8) lanes *= 2;
-        const int all = ((a.H + (k_pages ? a.G : 0)) * lanes + 31) / 32 * 32;
-        if (all <= 1024)
-            mm_launch(qk_prep_vec_kernel<TI, T, true>, dim3(n), dim3(all), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a, lanes);
-        else
-            mm_launch(qk_prep_vec_kernel<TI, T, false>, dim3(n), dim3(PREP_THREADS), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a, lanes);
-    } else {
+    int lanes = 1;
+    while (lanes < a.dk / 8) lanes *= 2;
+    const int all = ((a.H + (k_pages ? a.G : 0)) * lanes + 31) / 32 * 32;
+    // A lane for every unit of a row where a step's tokens have an SM to themselves (one such block fits an SM); with more tokens,
+    // smaller blocks side by side.  A 32-bit run keeps to the latter: its sums then have one order whatever else is in the step.
+    int turns = sizeof(T) == 2 && n <= 296 && all <= 1024 ? 1 : 2;
+    while (turns > 1 && turns < 8 && all > turns * PREP_THREADS) turns += turns < 4 ? 1 : 2;
+    if (!vec || all > 8 * PREP_THREADS) {
         mm_launch(qk_prep_kernel<TI, T>, dim3(n), dim3(PREP_THREADS), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a);
+        return;
     }
+    auto kernel = turns == 1 ? qk_prep_vec_kernel<TI, T, 1> : turns == 2 ? qk_prep_vec_kernel<TI, T, 2> : turns == 3 ? qk_prep_vec_kernel<TI, T, 3>
+                  : turns == 4 ? qk_prep_vec_kernel<TI, T, 4> : turns == 6 ? qk_prep_vec_kernel<TI, T, 6> : qk_prep_vec_kernel<TI, T, 8>;
+    // as few threads as the turns allow, so that none of them idles
+    const int threads = turns == 1 ? all : ((all + turns - 1) / turns + 31) / 32 * 32;
+    mm_launch(kernel, dim3(n), dim3(threads), 0, s, (const TI*)rows, (T*)q_out, (T*)k_pages, (T*)v_pages, a, lanes);
 }
 
 MM_EXPORT int mm_qk_prep(const void* rows, int rows_dtype, int ld, int q_off, int k_off, int v_off, const void* wq, const void* wk, float eps,

@@ -484,22 +484,34 @@ __global__ void attention_sink_merge_kernel(__nv_bfloat16* __restrict__ out, flo
                                             const float* __restrict__ part_ml, const int32_t* __restrict__ items, int H, int dv,
                                             int n_splits, int sink, const float* __restrict__ sink_logit, const float* __restrict__ gate,
                                             int gate_ld) {
+    __shared__ float factor[64];       // 2^(a split's maximum - the row's)
+    __shared__ float scale;
     const int item = blockIdx.x, h = blockIdx.y;
     const int t = items ? items[item] : item;
     const size_t p0 = ((size_t)item * H + h) * n_splits;
-    const bool with_sink = sink || sink_logit;
-    const float sink_m = sink_logit ? sink_logit[h] * SINK_LOG2E_F : 0.0f;
-    float m = with_sink ? sink_m : -INFINITY;
-    for (int s = 0; s < n_splits; ++s) m = fmaxf(m, part_ml[(p0 + s) * 2]);
-    const float mu = (m == -INFINITY) ? 0.0f : m;
-    float l = with_sink ? exp2f(sink_m - mu) : 0.0f;
-    for (int s = 0; s < n_splits; ++s) l += part_ml[(p0 + s) * 2 + 1] * exp2f(part_ml[(p0 + s) * 2] - mu);
-    const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * head_gate(gate, gate_ld, t, h);
+    if (threadIdx.x < 32) {            // one warp: a split per lane (at most 64)
+        const int lane = threadIdx.x;
+        const float2* ml = reinterpret_cast<const float2*>(part_ml) + p0;
+        const float2 none = make_float2(-INFINITY, 0.0f);
+        const float2 x = lane < n_splits ? ml[lane] : none, y = lane + 32 < n_splits ? ml[lane + 32] : none;
+        const bool with_sink = sink || sink_logit;
+        const float sink_m = sink_logit ? sink_logit[h] * SINK_LOG2E_F : 0.0f;
+        float m = warp_max(fmaxf(x.x, y.x));
+        if (with_sink) m = fmaxf(m, sink_m);
+        const float mu = (m == -INFINITY) ? 0.0f : m;
+        const float fx = exp2f(x.x - mu), fy = exp2f(y.x - mu);
+        const float l = warp_sum(x.y * fx + y.y * fy) + (with_sink ? exp2f(sink_m - mu) : 0.0f);
+        factor[lane] = fx;
+        factor[lane + 32] = fy;
+        if (lane == 0) scale = (l > 0.0f ? 1.0f / l : 0.0f) * head_gate(gate, gate_ld, t, h);
+    }
+    __syncthreads();
     for (int col = threadIdx.x; col < dv; col += blockDim.x) {
         float acc = 0.0f;
-        for (int s = 0; s < n_splits; ++s) acc += part_o[(p0 + s) * dv + col] * exp2f(part_ml[(p0 + s) * 2] - mu);
-        if (out32 != nullptr) out32[((size_t)t * H + h) * dv + col] = acc * inv;
-        else out[((size_t)t * H + h) * dv + col] = __float2bfloat16_rn(acc * inv);
+#pragma unroll 8
+        for (int s = 0; s < n_splits; ++s) acc = fmaf(part_o[(p0 + s) * dv + col], factor[s], acc);
+        if (out32 != nullptr) out32[((size_t)t * H + h) * dv + col] = acc * scale;
+        else out[((size_t)t * H + h) * dv + col] = __float2bfloat16_rn(acc * scale);
     }
 }
 

@@ -274,7 +274,7 @@ def test_a_readers_own_mask_over_anothers_keys(dtype, route):
 
 
 # ---- norms and rotation of queries and keys -----------------------------------------------------------------------------------
-@pytest.mark.parametrize("H,G,dk,dv,rot", [(4, 2, 64, 32, 64), (6, 3, 96, 64, 32), (3, 1, 9, 5, 6), (40, 8, 256, 128, 128), (2, 2, 24, 12, 24), (7, 7, 16, 3, 2), (5, 1, 40, 8, 0)])
+@pytest.mark.parametrize("H,G,dk,dv,rot", [(4, 2, 64, 32, 64), (6, 3, 96, 64, 32), (3, 1, 9, 5, 6), (40, 8, 256, 128, 128), (24, 8, 128, 16, 96), (16, 4, 128, 128, 128), (64, 8, 256, 8, 32), (2, 2, 24, 12, 24), (7, 7, 16, 3, 2), (5, 1, 40, 8, 0)])
 @pytest.mark.parametrize("scaling", [None, (8.0, 512, 32.0, 1.0)])
 def test_norms_and_rotation_far_out(H, G, dk, dv, rot, scaling):
     """Positions up to 500,000 turn as exactly as near ones; the norm over the whole projection, the unit norm after the rotation and
