@@ -259,16 +259,16 @@ def tupunex_latent_config(z):
 
 
 def nefelorn_config(z, experts=False):
-    """The four kinds of layers in turn: a window beside 4 kept tokens, runs of the window's length, the same with the keys and values of
+    """The four kinds of layers in turn: a window beside 8 kept tokens, runs of the window's length, the same with the keys and values of
     the layer before, a window again; every layer with a dense feed-forward, or (``experts``) with Domelix's routed experts (16 of
     three matrices, 4 chosen)."""
     d, expert_ff = z["width"], -(-(2 * z["ff"] // 12) // 64) * 64
     mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": 16, "top": 4, "scale": 2.0}} if experts else {"kind": "dense", "ff": z["ff"]}
     size = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5}
     far = dict(size, mask={"size": z["window"]},
-               rot={"base": 500000.0, "dims": z["dim"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+               rot={"base": 10000.0, "dims": z["dim"], "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
     near = {"type": "attention_2", "mlp": mlp,
-            "mixer": dict(size, mask={"size": z["window"], "keep_first": 4}, rot={"base": 500000.0, "dims": z["dim"] // 2})}
+            "mixer": dict(size, mask={"size": z["window"], "keep_first": 8}, rot={"base": 10000.0, "dims": z["dim"] // 2})}
     layers = [near if i % 4 in (0, 3) else {"type": "attention", "mlp": mlp, "mixer": far if i % 4 == 1 else dict(far, kv_from=i - 1)}
               for i in range(z["layers"])]
     return {"architecture": "Nefelorn", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "logit_softcap": 30.0,

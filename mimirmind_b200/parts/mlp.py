@@ -111,6 +111,8 @@ class SwiGLU(FeedForward):
 # step of 8 layers: width 4096 / ff 16384: 4.68 against 4.71 ms; width 2048 / ff 8192: 2.46 against 2.20 ms, where the
 # step is bound by launching and the tensor maps of every call cost host time).
 FUSED_UP_MIN_HIDDEN = 4096
+# The exact gelu as a pass of its own takes longer (width 2048 / ff 8192: product 51 + pass 25 us against 67 us in one).
+FUSED_UP_MIN_HIDDEN_OF = {"gelu_erf": 2048}
 
 
 @FEED_FORWARDS.register("dense_mlp")
@@ -158,7 +160,7 @@ class DenseMLP(FeedForward):
             # a few tokens: bias and activation in the epilogue of the weight-streaming product
             return ops.gemv_bf16_act(x, self.w_up, self.b_up, self.activation)
         if (x.dtype == torch.bfloat16 and self.w_up.dtype == torch.bfloat16 and self.rt.matmul != "simt" and not ctx.plain_only
-                and x.shape[0] >= ops.TCGEN05_SWIGLU_MIN_ROWS and self.hidden >= FUSED_UP_MIN_HIDDEN
+                and x.shape[0] >= ops.TCGEN05_SWIGLU_MIN_ROWS and self.hidden >= FUSED_UP_MIN_HIDDEN_OF.get(self.activation, FUSED_UP_MIN_HIDDEN)
                 and ops.gemm_tcgen05_supported(x.shape[0], self.ff, self.hidden)):
             # prompt-sized and deep enough: the tcgen05 product with bias and activation as its epilogue (the hidden rows
             # never exist without their activation), as the gated feed-forward does with SwiGLU
